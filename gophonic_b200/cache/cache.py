@@ -36,7 +36,7 @@ from typing import Dict, List, Optional, Sequence, Tuple
 import numpy as np
 import torch
 
-from ..parts.base import KVRequest, KVStateRequest, StateRequest
+from ..parts.base import BlockStateRequest, KVRequest, KVStateRequest, StateRequest
 
 PAGE = 64
 
@@ -115,6 +115,14 @@ class StateView:
 
 
 @dataclass
+class BlockView:
+    """The view of a run whose block keeps a state of its own beside its mixer's cache."""
+    mixer: object              # what the mixer asked for: a KVView, a StateView or None
+    state: torch.Tensor        # [max_slots, *shape]
+    writable: bool = True
+
+
+@dataclass
 class CacheMark:
     """What ``Cache.snapshot`` returns: a length and the state of that moment."""
     slot: int
@@ -152,9 +160,18 @@ class Cache:
         self._state_groups: Dict[Tuple[Tuple[int, ...], torch.dtype], List[int]] = {}
         self._plane: Dict[int, Tuple[str, object, int]] = {}
         self._beside: Dict[int, Tuple[object, int]] = {}     # the state plane of a run that asked for keys and state
+        self._of_block: Dict[int, Tuple[object, int]] = {}   # the state plane of a run whose block asked for one
         self._cache_of: Dict[int, Optional[int]] = {}
         for pos, (req, cache_of) in enumerate(requests):
             self._cache_of[pos] = cache_of
+            if isinstance(req, BlockStateRequest):
+                if cache_of is not None:
+                    raise CacheError(f"schedule position {pos}: a run whose block keeps a state cannot read another run's cache")
+                key = (tuple(req.state.shape), req.state.dtype)
+                planes = self._state_groups.setdefault(key, [])
+                self._of_block[pos] = (key, len(planes))
+                planes.append(pos)
+                req = req.mixer
             if cache_of is not None or req is None:
                 continue
             if isinstance(req, KVStateRequest):
@@ -233,6 +250,12 @@ class Cache:
 
     def view(self, pos: int):
         """The cache view of schedule position ``pos`` (None if it asked for nothing)."""
+        if pos in self._of_block:
+            key, ordinal = self._of_block[pos]
+            return BlockView(self._mixer_view(pos), self._state[key][ordinal])
+        return self._mixer_view(pos)
+
+    def _mixer_view(self, pos: int):
         src = self._cache_of.get(pos)
         writable = src is None
         at = pos if src is None else src

@@ -32,6 +32,25 @@ class RMSNormSpec:
 
 
 @dataclass(frozen=True)
+class LinearStretch:
+    """``scaling`` of a rotation: every frequency is divided by ``factor``."""
+    factor: float
+
+
+@dataclass(frozen=True)
+class RampStretch:
+    """``scaling`` of a rotation over ``dims`` channels with base b, blended along the channels (YaRN).  The channel
+    pair whose wave turns t times in ``original`` positions has the number c(t) = dims ln(original / (2 pi t)) / (2 ln b).
+    Pairs below floor(c(fast)) keep their frequency, pairs above ceil(c(slow)) have it divided by ``factor``, and between
+    the two (clamped to 0 and dims - 1) a straight line in the pair's number blends the divided and the plain one.  Cosines and
+    sines are multiplied by 0.1 ln(factor) + 1."""
+    factor: float
+    original: float
+    fast: float
+    slow: float
+
+
+@dataclass(frozen=True)
 class RotarySpec:
     """Rotate-half rotary embedding over the first ``rotary_dim`` elements of each head.
 
@@ -41,13 +60,14 @@ class RotarySpec:
     ``scaling`` = (factor, low, high, original) stretches the slow frequencies for contexts longer than
     ``original`` positions: a frequency f whose wavelength 2 pi / f is longer than original / low becomes
     f / factor, one whose wavelength is shorter than original / high stays, and in between
-    s = (original / wavelength - low) / (high - low) blends them as (1 - s) f / factor + s f.
+    s = (original / wavelength - low) / (high - low) blends them as (1 - s) f / factor + s f.  It may also be a
+    ``LinearStretch`` or a ``RampStretch``.
     """
     head_dim: int
     rotary_dim: int
     theta: float
     kind: str = "rope"
-    scaling: Optional[Tuple[float, float, float, float]] = None
+    scaling: Optional[object] = None
 
 
 @dataclass(frozen=True)
@@ -59,7 +79,7 @@ class PairRotarySpec:
     rotary_dim: int
     theta: float
     kind: str = "rope_pairs"
-    scaling: Optional[Tuple[float, float, float, float]] = None
+    scaling: Optional[object] = None
 
 
 @dataclass(frozen=True)
@@ -100,7 +120,11 @@ class GatedAttentionSpec:
     * ``qk_norm`` (an ``RMSNormSpec`` whose eps is used): q and k are RMS-normed after their biases and before the
       position encoding; with ``qk_norm_span`` over the whole projection at once (all heads of q share one mean of
       squares and a weight of heads * head_dim, tensor ``q.norm``; k likewise), else head by head with a weight
-      of head_dim;
+      of head_dim.  ``qk_norm_weight`` False: a norm without a weight (no tensors); ``qk_norm_after``: the norm stands
+      behind the position encoding (only without a weight, and with an encoding that keeps a head's length: then the
+      two orders are the same function, since a rotation changes no sum of squares);
+    * ``value_from_key``: there is no value projection, the values are the keys as projected, before norm and rotation
+      (``value_dim`` = ``head_dim``);
     * ``out_bias``: the output projection carries a bias too;
     * ``gate``: the concatenated heads are multiplied by sigmoid of a further projection of the
       mixer's input before the output projection;
@@ -126,6 +150,9 @@ class GatedAttentionSpec:
     qk_norm: Optional[RMSNormSpec] = None
     qk_norm_span: bool = False
     out_bias: bool = False
+    qk_norm_weight: bool = True
+    qk_norm_after: bool = False
+    value_from_key: bool = False
     names: Tuple[Tuple[str, str], ...] = (("q", "q"), ("k", "k"), ("v", "v"), ("g", "g"), ("o", "o"), ("q_norm", "q.norm"),
                                           ("k_norm", "k.norm"), ("sink", "sink"))
     bias_suffix: str = ".b"
@@ -173,7 +200,8 @@ class LatentAttentionSpec:
         per head: k = [W_uk c | k_r],  v = W_uv c  (value_dim),   score = (q . k) * scale
 
     Only c and k_r are cached.  ``position`` is the encoding of the rotated part (its ``head_dim`` is rot_dim);
-    ``window`` > 0: row i sees j with 0 <= i - j < window; ``chunk`` > 0: only its own block of positions."""
+    ``window`` > 0: row i sees j with 0 <= i - j < window; ``chunk`` > 0: only its own block of positions.  ``gate``: the
+    concatenated heads are multiplied by sigmoid(W_g h) ahead of the output projection."""
     hidden: int
     heads: int
     head_dim: int
@@ -186,8 +214,9 @@ class LatentAttentionSpec:
     eps: float
     window: int = 0
     chunk: int = 0
+    gate: bool = False
     names: Tuple[Tuple[str, str], ...] = (("dq", "dq"), ("dq_norm", "dq.norm"), ("uq", "uq"), ("dkv", "dkv"), ("dkv_norm", "dkv.norm"),
-                                          ("uk", "uk"), ("uv", "uv"), ("o", "o"))
+                                          ("uk", "uk"), ("uv", "uv"), ("g", "g"), ("o", "o"))
     kind: str = "latent_attention"
 
 
@@ -248,6 +277,25 @@ class DeltaRuleSpec:
 
 
 @dataclass(frozen=True)
+class ForgetStateSpec:
+    """HGRN2: linear attention whose forget gate also decides what is written.  Per head a matrix state S (key_dim x
+    value_dim, float32), with q = silu(W_q x), v = W_v x and per key channel
+    f = l + (1 - l) sigmoid(W_f x + b), l a learned lower bound:
+
+        S <- diag(f) S + (1 - f) v^T,   o = S^T q.
+
+    Each head's o is RMS-normed with one weight of ``value_dim`` shared by the heads, and projected back.  ``names`` maps
+    q, v, f, the gate's bias, the lower bound, the norm's weight and the output projection to tensor-name suffixes."""
+    hidden: int
+    heads: int
+    key_dim: int
+    value_dim: int
+    eps: float
+    names: Tuple[Tuple[str, str], ...] = (("q", "q"), ("v", "v"), ("f", "f"), ("f_bias", "f.b"), ("lower", "lower"), ("norm", "norm"), ("o", "o"))
+    kind: str = "hgrn2"
+
+
+@dataclass(frozen=True)
 class SigmoidAttentionSpec:
     """Grouped-query attention whose weights are not normalised over the keys: a visible key j weighs
     sigmoid((q_i . k_j) * scale + b_h), with b_h one number per head (``score_bias``).  Options:
@@ -295,7 +343,11 @@ class MoESpec:
     * ``shared``: the spec of a further feed-forward under ``shared_prefix`` that every token uses, with weight 1, or
       with ``shared_gate`` with weight sigmoid(w . x), w the tensor ``shared_prefix + shared_gate_name`` ([1, hidden]);
     * ``router_bias``: the router's logits carry a bias (tensor ``router`` + ``router_bias_suffix``);
-    * ``renorm_eps`` 0 with ``score`` "softmax" and ``renorm``: the weights are the softmax over the chosen logits alone."""
+    * ``renorm_eps`` 0 with ``score`` "softmax" and ``renorm``: the weights are the softmax over the chosen logits alone;
+    * ``correction``: an expert is chosen by its score plus a learned number (tensor ``correction_name``, one an expert);
+      the weights come from the score without it;
+    * ``groups`` > 1: the experts form that many equal groups of neighbours, a group counts as the sum of its two largest
+      choice scores, and only experts of the ``keep_groups`` best groups can be chosen."""
     hidden: int
     experts: int
     top: int
@@ -314,6 +366,10 @@ class MoESpec:
     router_bias_suffix: str = ".b"
     shared_gate: bool = False
     shared_gate_name: str = "sg"
+    correction: bool = False
+    correction_name: str = "correction"
+    groups: int = 1
+    keep_groups: int = 1
 
 
 @dataclass(frozen=True)
@@ -419,6 +475,40 @@ class PostNormLayerSpec:
 
 
 @dataclass(frozen=True)
+class SandwichLayerSpec:
+    """One layer with a norm in front of and behind each sublayer:
+
+        x <- x + out_norm_1(mixer(h)),   h = norm_1(x);     x <- x + out_norm_2(feed_forward(norm_2(x)))
+
+    * ``conv_taps`` > 0: what the mixer reads passes a causal convolution over time on each channel that is added to it,
+      h_t <- h_t + sum_j w[:, j] h_(t - taps + 1 + j) (tensor ``conv_name``, [width, taps]; zeros before the start); a
+      sequence's last taps - 1 rows h are part of its state;
+    * ``average``: with X_0 the embedding output and X_(i+1) the result of the layer that runs at place i of the schedule,
+      what goes on behind it is sum over j = 0 .. i+1 of w[j] X_j (tensor ``average_name``, [i + 2]; ``average`` is that
+      length, 0: the result itself goes on).
+
+    ``feed_forward`` None (with its two norms): the layer is its mixer sublayer alone."""
+    prefix: str
+    mixer: object
+    feed_forward: object
+    mixer_norm: object
+    mixer_out_norm: object
+    feed_forward_norm: object
+    feed_forward_out_norm: object
+    conv_taps: int = 0
+    average: int = 0
+    block: str = "sandwich"
+    mixer_prefix: str = "mix."
+    feed_forward_prefix: str = "mlp."
+    mixer_norm_prefix: str = "norm1"
+    mixer_out_norm_prefix: str = "norm1b"
+    feed_forward_norm_prefix: str = "norm2"
+    feed_forward_out_norm_prefix: str = "norm2b"
+    conv_name: str = "canon1"
+    average_name: str = "dwa"
+
+
+@dataclass(frozen=True)
 class ReinjectSpec:
     """What happens to the residual where a pass through repeated layers begins: with the embedding output x0,
 
@@ -462,11 +552,13 @@ class EmbeddingSpec:
 @dataclass(frozen=True)
 class HeadSpec:
     """Output projection hidden -> vocab.  If the checkpoint has no tensor ``name`` the head is
-    tied to ``tied_to`` (qwen3/chat.go:55-65 decides by tensor presence, never by a flag)."""
+    tied to ``tied_to`` (qwen3/chat.go:55-65 decides by tensor presence, never by a flag).
+    ``soft_cap`` > 0: the logits become soft_cap * tanh(logits / soft_cap)."""
     name: str
     vocab: int
     hidden: int
     tied_to: Optional[str] = None
+    soft_cap: float = 0.0
 
 
 @dataclass(frozen=True)

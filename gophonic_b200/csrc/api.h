@@ -82,6 +82,7 @@ struct QkRopeParamsX : QkRopeParams {
     int dv;            // size of a value head; 0: the same as d
     int span;          // 1: q is normed over all its heads together (q_w: [heads * d]) and k likewise (k_w: [kv_heads * d]); 0: per head
     int v_share;       // > 1: the row holds kv_heads / v_share value heads (that many key heads read one value head); 0, 1: kv_heads
+    int v_from_k;      // 1: the row holds no value heads; a value is its key as it stands in the row, before norm and rotation
 };
 
 // A matrix state per (sequence, head), updated token by token: S <- diag(a) S + b k v^T, o = S^T q.
@@ -108,6 +109,9 @@ struct LinearStateParams {
     int scalar_decay;
     int max_slots;
     int max_q_len;          // most rows a sequence brings; 1 selects the kernel for single tokens
+    const float* lower;     // not null: the forget gate also writes.  decay holds its pre-activations z (gate_bias [heads * d] is added);
+                            // u = (1 - lower) sigmoid(-z), S <- S + u (v - S), o = S^T silu(q); float32 rows; [heads * d]
+    int rows;               // rows of qkv
 };
 
 // y = norm(x / divisor) * weight * gate(g) per (row, head); one warp a head.
@@ -124,7 +128,7 @@ struct HeadGateParams {
     int weight_per_head;
     int normed;             // 1: x over its root mean square (eps under the root) first
     float eps;
-    int gate_kind;          // 0: sigmoid(g); 1: g * sigmoid(g)
+    int gate_kind;          // 0: sigmoid(g); 1: g * sigmoid(g); 2: no gate (gate is null)
     int rows, heads, size;
 };
 
@@ -303,6 +307,9 @@ struct MoeRouteParams {
     float* weight;          // [rows, top]
     int score_kind;         // 0: softmax over all experts; 1: sigmoid of each logit by itself
     int renorm;             // 1: the chosen scores are divided by their sum + renorm_eps; 0: they are the weights
+    const float* correction;   // [experts] added to the scores for the choice alone, or null
+    int groups, keep_groups;   // groups > 1: equal groups of neighbours; only experts of the keep_groups best ones (sum of a group's
+                               // two largest choice scores) can be chosen
 };
 GB_API int gb_moe_route(const MoeRouteParams* p, cudaStream_t stream);
 GB_API int gb_moe_act(const void* up, int64_t up_stride, const float* dense, void* act, int64_t act_stride, int rows, int experts, int ff,
@@ -354,3 +361,34 @@ GB_API int gb_head_gemm_mma(const void* a, int64_t a_row_stride, int64_t a_head_
                             int64_t o_head_stride, int rows, int heads, int K, int N, cudaStream_t stream);
 GB_API int gb_head_gemm(const void* a, int64_t a_row_stride, int64_t a_head_stride, const void* w, void* out, int64_t o_row_stride,
                         int64_t o_head_stride, int rows, int heads, int K, int N, int dtype, int w_dtype, cudaStream_t stream);
+
+// Blocks with norms on both sides of a sublayer, a short convolution and a weighted sum over the depth (sandwich.cu).
+struct SandwichParams {
+    const float* base;      // [rows, width]
+    const float* y;         // [rows, width] or null: v = base + y / rms(y) * y_w
+    const float* y_w;
+    float y_eps;
+    float* result;          // v is stored here, or null
+    const float* planes;    // [n_planes, ...]: x = sum_j average[j] planes[j] + average[n_planes] v; average null: x = v
+    int64_t plane_stride;
+    int n_planes;
+    const float* average;
+    float* x_out;           // x is stored here, or null
+    const float* norm_w;    // out = x / rms(x) * norm_w
+    float norm_eps;
+    void* out;
+    const int* row_index;   // out row i is made from row row_index[i], or null
+    const float* conv_w;    // [taps, width] or null: every row is its sequence's single token and is convolved on its way out
+    int taps;
+    float* state;           // [slots, state_slot_stride]: the sequence's last taps - 1 normed rows, oldest first
+    int64_t state_slot_stride;
+    const int* row_seq;
+    const int* seq_slot;
+    int max_slots;
+    int rows, width;
+};
+GB_API int gb_sandwich_rows(const SandwichParams* p, int out_dtype, cudaStream_t stream);
+GB_API int gb_conv_rows(const float* h, const float* conv_w, int taps, float* state, int64_t state_slot_stride, int max_slots, void* out, int out_dtype,
+                        int rows, int width, int nseq, const int* row_seq, const int* seq_slot, const int* seq_q_start, const int* seq_q_len,
+                        cudaStream_t stream);
+GB_API int gb_soft_cap(float* z, int64_t n, float cap, cudaStream_t stream);

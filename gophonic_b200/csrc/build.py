@@ -54,6 +54,7 @@ SOURCES = [
     "moe.cu",
     "postnorm.cu",
     "attention_latent.cu",
+    "sandwich.cu",
     "sampling.cu",
     "no_alloc.cu",
     "dispatch.cu",

@@ -362,7 +362,8 @@ __global__ void qk_rope_kernel(QkRopeParamsX p) {
     int kvh = is_q ? 0 : (is_k ? head - p.heads : head - p.heads - p.kv_heads);
     // q and k heads are d wide, the value heads behind them dv
     T* src = (T*)p.qkv + (int64_t)r * p.row_stride +
-             (is_q || is_k ? (int64_t)head * d : (int64_t)(p.heads + p.kv_heads) * d + (int64_t)kvh * dv);
+             (is_q || is_k ? (int64_t)head * d
+                           : (p.v_from_k ? (int64_t)(p.heads + kvh) * d : (int64_t)(p.heads + p.kv_heads) * d + (int64_t)kvh * dv));
     const float* bias = is_q ? p.q_b : (is_k ? p.k_b : p.v_b);
     if (bias) bias += (is_q ? head : kvh) * (is_q || is_k ? d : dv);
 
@@ -651,7 +652,7 @@ __global__ void __launch_bounds__(256) qk_rope_span_vec_kernel(QkRopeParamsX p) 
 // and it takes several in flight per thread to keep the memory system busy.
 constexpr int ROPE_ROWS = 4;
 
-__global__ void __launch_bounds__(256) qk_rope_bf16_d128_kernel(QkRopeParams p) {
+__global__ void __launch_bounds__(256) qk_rope_bf16_d128_kernel(QkRopeParams p, int v_from_k) {
     pdl_wait();
     pdl_trigger();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -666,6 +667,8 @@ __global__ void __launch_bounds__(256) qk_rope_bf16_d128_kernel(QkRopeParams p) 
     const int kvh = is_q ? 0 : (is_k ? head - p.heads : head - p.heads - p.kv_heads);
     const float* w = is_q ? p.q_w : p.k_w;
     const int ci = (lane & 15) * 4;  // index into the 64 angles of a position
+    // the head's place in the row: a value that is a key is read where the key stands (keys are not changed in the row)
+    const int column = v_from_k && !is_q && !is_k ? head - p.kv_heads : head;
 
     int pos[ROPE_ROWS];
     uint2 raw[ROPE_ROWS];
@@ -675,7 +678,7 @@ __global__ void __launch_bounds__(256) qk_rope_bf16_d128_kernel(QkRopeParams p) 
     for (int j = 0; j < ROPE_ROWS; j++) {
         const int r = r0 + j < p.rows ? r0 + j : p.rows - 1;  // rows past the end repeat the last one and are not stored
         pos[j] = p.row_pos[r];
-        bf* src = (bf*)p.qkv + (int64_t)r * p.row_stride + (int64_t)head * 128 + lane * 4;
+        bf* src = (bf*)p.qkv + (int64_t)r * p.row_stride + (int64_t)column * 128 + lane * 4;
         raw[j] = *reinterpret_cast<const uint2*>(src);
         dst[j] = src;
     }
@@ -742,7 +745,7 @@ __global__ void __launch_bounds__(256) qk_rope_bf16_d128_kernel(QkRopeParams p) 
 // two heads of WIDE_ROWS consecutive rows.
 constexpr int WIDE_ROWS = 4;
 
-__global__ void __launch_bounds__(256) qk_rope_bf16_d128_wide_kernel(QkRopeParams p) {
+__global__ void __launch_bounds__(256) qk_rope_bf16_d128_wide_kernel(QkRopeParams p, int v_from_k) {
     pdl_wait();
     pdl_trigger();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, l16 = lane & 15;
@@ -758,6 +761,7 @@ __global__ void __launch_bounds__(256) qk_rope_bf16_d128_wide_kernel(QkRopeParam
     const int kvh = is_q ? 0 : (is_k ? head - p.heads : head - p.heads - p.kv_heads);
     const float* w = is_q ? p.q_w : p.k_w;
     const int ci = (l16 & 7) * 8;  // index into the 64 angles of a position
+    const int column = v_from_k && !is_q && !is_k ? head - p.kv_heads : head;
 
     int pos[WIDE_ROWS];
     uint4 raw[WIDE_ROWS];
@@ -766,7 +770,7 @@ __global__ void __launch_bounds__(256) qk_rope_bf16_d128_wide_kernel(QkRopeParam
     for (int j = 0; j < WIDE_ROWS; j++) {
         const int r = r0 + j < p.rows ? r0 + j : p.rows - 1;  // rows past the end repeat the last one and are not stored
         pos[j] = p.row_pos[r];
-        bf* src = (bf*)p.qkv + (int64_t)r * p.row_stride + (int64_t)head * 128 + l16 * 8;
+        bf* src = (bf*)p.qkv + (int64_t)r * p.row_stride + (int64_t)column * 128 + l16 * 8;
         raw[j] = *reinterpret_cast<const uint4*>(src);
         dst[j] = src;
     }
@@ -832,7 +836,7 @@ GB_API int gb_qk_norm_rope_kv_write(const QkRopeParams* pp, int dtype, cudaStrea
     QkRopeParamsX x;
     static_cast<QkRopeParams&>(x) = *pp;
     x.q_b = x.k_b = x.v_b = nullptr;
-    x.pairs = x.dv = x.span = x.v_share = 0;
+    x.pairs = x.dv = x.span = x.v_share = x.v_from_k = 0;
     return gb_qk_norm_rope_kv_write_x(&x, dtype, stream);
 }
 
@@ -847,6 +851,8 @@ GB_API int gb_qk_norm_rope_kv_write_x(const QkRopeParamsX* pp, int dtype, cudaSt
     if (p.v_share < 0 || (p.v_share > 1 && p.kv_heads % p.v_share)) GB_REFUSE("qk_norm_rope: %d key heads share value heads by %d", p.kv_heads, p.v_share);
     int total_heads = p.heads + p.kv_heads + (p.v_share > 1 ? p.kv_heads / p.v_share : p.kv_heads);
     if (p.dv < 0 || p.dv > 1024) GB_REFUSE("qk_norm_rope: value size %d is outside [1, 1024]", p.dv);
+    if (p.v_from_k && (p.span || p.v_share > 1 || p.q_b || p.k_b || p.v_b || (p.dv != 0 && p.dv != p.d)))
+        GB_REFUSE("qk_norm_rope: values that are the keys are as many and as wide as they are, without biases and without a norm over all heads");
     if (p.span && p.v_share > 1) GB_REFUSE("qk_norm_rope: shared value heads with a norm over all heads are not built");
     if (p.span) {
         const size_t span_smem = ((size_t)(p.heads + p.kv_heads) * p.d + 16) * sizeof(float);
@@ -879,11 +885,11 @@ GB_API int gb_qk_norm_rope_kv_write_x(const QkRopeParamsX* pp, int dtype, cudaSt
         // prompts: the kernel of 16-byte accesses (it adds a row's squares up in another order, so a key
         // may differ in its last bit from the one the kernel for few rows would write)
         if (p.rows >= 256 && !(p.row_stride & 7) && !((uintptr_t)p.qkv & 15)) {
-            launch_pdl(qk_rope_bf16_d128_wide_kernel, dim3(ceil_div(p.rows, WIDE_ROWS), ceil_div(total_heads, 16)), dim3(256), 0, stream, p);
+            launch_pdl(qk_rope_bf16_d128_wide_kernel, dim3(ceil_div(p.rows, WIDE_ROWS), ceil_div(total_heads, 16)), dim3(256), 0, stream, p, p.v_from_k);
             GB_CHECK_LAUNCH("qk_norm_rope_kv_write");
             return 0;
         }
-        launch_pdl(qk_rope_bf16_d128_kernel, dim3(ceil_div(p.rows, ROPE_ROWS), ceil_div(total_heads, 8)), dim3(256), 0, stream, p);
+        launch_pdl(qk_rope_bf16_d128_kernel, dim3(ceil_div(p.rows, ROPE_ROWS), ceil_div(total_heads, 8)), dim3(256), 0, stream, p, p.v_from_k);
         GB_CHECK_LAUNCH("qk_norm_rope_kv_write");
         return 0;
     }

@@ -41,6 +41,26 @@ __global__ void gla_decay_kernel(float* __restrict__ z, const float* __restrict_
 }
 
 // ------------------------------------------------------------------------------------------
+// The forget gate that also writes (HGRN2), in place on float32 rows, two channels' worth of work a thread:
+// q <- silu(q) and z <- u = (1 - l) sigmoid(-(z + bias)), the write gate 1 - f of f = l + (1 - l) sigmoid(z + bias)
+// (formed this way it keeps its digits where f is close to one).
+__device__ __forceinline__ float write_gate(float z, float bias, float low) { return (1.f - low) / (1.f + expf(z + bias)); }
+__device__ __forceinline__ float silu_f32(float x) { return x / (1.f + expf(-x)); }
+
+__global__ void forget_gate_kernel(float* __restrict__ q, int64_t q_stride, float* __restrict__ z, int64_t z_stride, const float* __restrict__ bias,
+                                   const float* __restrict__ lower, int64_t total, int width) {
+    const int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x;
+    if (i >= total) return;
+    const int64_t r = i / width;
+    const int c = (int)(i % width);
+    float* qp = q + r * q_stride + c;
+    float* zp = z + r * z_stride + c;
+    const float x = *qp, y = *zp;
+    *qp = silu_f32(x);
+    *zp = write_gate(y, bias ? bias[c] : 0.f, lower[c]);
+}
+
+// ------------------------------------------------------------------------------------------
 // gates of the matrix memory.  One warp per (sequence, head), 32 tokens at a time: the lanes take a
 // token each for the capped gates, the running maximum m_t = max(f_t + m_(t-1), i_t) is walked in
 // order through shuffles (an add and a max a token), then the lanes turn their token's values into
@@ -87,15 +107,17 @@ __global__ void __launch_bounds__(32) mlstm_gates_kernel(LinearStateParams p) {
 }
 
 // ------------------------------------------------------------------------------------------
-// the scan.  RC: key channels per slice (a multiple of 4, RC * 8 >= d).  SCALAR: one decay per head
+// the scan.  RC: key channels per slice (a multiple of 4, RC * 8 >= d).  MODE 1: one decay per head
 // and token (coef), with the input gate folded into the staged keys and one more block of columns
-// for the normaliser; otherwise a decay per key channel (p.decay).
-template <typename T, int RC, bool SCALAR>
+// for the normaliser; MODE 0: a decay per key channel (p.decay); MODE 2: a write gate u per key channel
+// (p.decay), S <- S + u (v - S), with no key: one staged row less and the same arithmetic an element.
+template <typename T, int RC, int MODE>
 __global__ void __launch_bounds__(THREADS) state_scan_kernel(LinearStateParams p) {
+    constexpr bool SCALAR = MODE == 1, WRITES = MODE == 2;
     constexpr int P = (RC / 4) % 2 ? RC : RC + 4;   // slice stride in floats: P / 4 odd, so the 8 slices' 16-byte reads miss each other's banks
     constexpr int ROW = SLICES * P;
     __shared__ __align__(16) float q_s[TT][ROW];
-    __shared__ __align__(16) float k_s[TT][ROW];
+    __shared__ __align__(16) float k_s[WRITES ? 1 : TT][WRITES ? 4 : ROW];
     __shared__ __align__(16) float a_s[SCALAR ? 1 : TT][SCALAR ? 4 : ROW];
     __shared__ float v_s[TT][COLS];
     __shared__ float o_s[TT][COLS];
@@ -166,7 +188,7 @@ __global__ void __launch_bounds__(THREADS) state_scan_kernel(LinearStateParams p
             const int64_t row = q_start + t0 + t;
             const T* r = base + row * p.row_stride;
             rq[e] = r[p.q_off + h * d + c];
-            rk[e] = r[p.k_off + h * d + c];
+            if (!WRITES) rk[e] = r[p.k_off + h * d + c];
             ra[e] = SCALAR ? p.coef[(row * H + h) * 4 + 1] : p.decay[row * p.decay_stride + h * d + c];
         }
         {
@@ -193,8 +215,8 @@ __global__ void __launch_bounds__(THREADS) state_scan_kernel(LinearStateParams p
             const bool there = t < nt && c < d;
             q_s[t][at] = there ? to_f32<T>(rq[e]) * p.q_scale : 0.f;
             // one decay per head: the input gate goes into the key, the decay itself is keep_s
-            k_s[t][at] = there ? (SCALAR ? to_f32<T>(rk[e]) * ra[e] : to_f32<T>(rk[e])) : 0.f;
-            if (!SCALAR) a_s[t][at] = there ? ra[e] : 1.f;
+            if (!WRITES) k_s[t][at] = there ? (SCALAR ? to_f32<T>(rk[e]) * ra[e] : to_f32<T>(rk[e])) : 0.f;
+            if (!SCALAR) a_s[t][at] = there ? ra[e] : (WRITES ? 0.f : 1.f);
         }
         {
             const int t = tid / COLS, jj = tid % COLS;
@@ -225,13 +247,21 @@ __global__ void __launch_bounds__(THREADS) state_scan_kernel(LinearStateParams p
 #pragma unroll
             for (int i = 0; i < RC; i += 4) {
                 const float4 q4 = *reinterpret_cast<const float4*>(&q_s[t][slice * P + i]);
-                const float4 k4 = *reinterpret_cast<const float4*>(&k_s[t][slice * P + i]);
+                float4 k4 = make_float4(0.f, 0.f, 0.f, 0.f);
+                if (!WRITES) k4 = *reinterpret_cast<const float4*>(&k_s[t][slice * P + i]);
                 float4 a4 = make_float4(keep, keep, keep, keep);
                 if (!SCALAR) a4 = *reinterpret_cast<const float4*>(&a_s[t][slice * P + i]);
-                st[i] = fmaf(a4.x, st[i], k4.x * vj);
-                st[i + 1] = fmaf(a4.y, st[i + 1], k4.y * vj);
-                st[i + 2] = fmaf(a4.z, st[i + 2], k4.z * vj);
-                st[i + 3] = fmaf(a4.w, st[i + 3], k4.w * vj);
+                if (WRITES) {
+                    st[i] = fmaf(a4.x, vj - st[i], st[i]);
+                    st[i + 1] = fmaf(a4.y, vj - st[i + 1], st[i + 1]);
+                    st[i + 2] = fmaf(a4.z, vj - st[i + 2], st[i + 2]);
+                    st[i + 3] = fmaf(a4.w, vj - st[i + 3], st[i + 3]);
+                } else {
+                    st[i] = fmaf(a4.x, st[i], k4.x * vj);
+                    st[i + 1] = fmaf(a4.y, st[i + 1], k4.y * vj);
+                    st[i + 2] = fmaf(a4.z, st[i + 2], k4.z * vj);
+                    st[i + 3] = fmaf(a4.w, st[i + 3], k4.w * vj);
+                }
                 acc0 = fmaf(st[i], q4.x, acc0);
                 acc1 = fmaf(st[i + 1], q4.y, acc1);
                 acc2 = fmaf(st[i + 2], q4.z, acc2);
@@ -300,12 +330,13 @@ __global__ void __launch_bounds__(THREADS) state_scan_kernel(LinearStateParams p
 // lane its own 16 bytes, no two quarter-warps the same bytes), four times less shared-memory traffic
 // than with 8 slices and a column a thread, for the same registers.  A tile's 8 tokens x 4 columns of
 // sums are added up over the 32 slices by a five-step exchange that leaves each lane one of them.
-template <typename T, int RC, bool SCALAR>
+template <typename T, int RC, int MODE>
 __global__ void __launch_bounds__(THREADS) state_scan_wide_kernel(LinearStateParams p) {
+    constexpr bool SCALAR = MODE == 1, WRITES = MODE == 2;
     constexpr int D = 32 * RC;          // key channels of a head
     constexpr int CW = 4;               // columns a warp (and a thread) owns
     __shared__ __align__(16) float q_s[TT][D];
-    __shared__ __align__(16) float k_s[TT][D];
+    __shared__ __align__(16) float k_s[WRITES ? 1 : TT][WRITES ? 4 : D];
     __shared__ __align__(16) float a_s[SCALAR ? 1 : TT][SCALAR ? 4 : D];
     __shared__ __align__(16) float v_s[TT][COLS];
     __shared__ float o_s[TT][COLS];
@@ -367,7 +398,7 @@ __global__ void __launch_bounds__(THREADS) state_scan_wide_kernel(LinearStatePar
             const int64_t row = q_start + t0 + t;
             const T* r = base + row * p.row_stride;
             rq[e] = r[p.q_off + h * D + c];
-            rk[e] = r[p.k_off + h * D + c];
+            if (!WRITES) rk[e] = r[p.k_off + h * D + c];
             ra[e] = SCALAR ? p.coef[(row * H + h) * 4 + 1] : p.decay[row * p.decay_stride + h * D + c];
         }
         {
@@ -392,8 +423,8 @@ __global__ void __launch_bounds__(THREADS) state_scan_wide_kernel(LinearStatePar
             const int t = idx / D, c = idx % D;
             const bool there = t < nt;
             q_s[t][c] = there ? to_f32<T>(rq[e]) * p.q_scale : 0.f;
-            k_s[t][c] = there ? (SCALAR ? to_f32<T>(rk[e]) * ra[e] : to_f32<T>(rk[e])) : 0.f;
-            if (!SCALAR) a_s[t][c] = there ? ra[e] : 1.f;
+            if (!WRITES) k_s[t][c] = there ? (SCALAR ? to_f32<T>(rk[e]) * ra[e] : to_f32<T>(rk[e])) : 0.f;
+            if (!SCALAR) a_s[t][c] = there ? ra[e] : (WRITES ? 0.f : 1.f);
         }
         {
             const int t = tid / COLS, jj = tid % COLS;
@@ -422,7 +453,8 @@ __global__ void __launch_bounds__(THREADS) state_scan_wide_kernel(LinearStatePar
 #pragma unroll
             for (int i = 0; i < RC; i += 4) {
                 const float4 q4 = *reinterpret_cast<const float4*>(&q_s[t][lane * RC + i]);
-                const float4 k4 = *reinterpret_cast<const float4*>(&k_s[t][lane * RC + i]);
+                float4 k4 = make_float4(0.f, 0.f, 0.f, 0.f);
+                if (!WRITES) k4 = *reinterpret_cast<const float4*>(&k_s[t][lane * RC + i]);
                 float4 a4 = make_float4(keep, keep, keep, keep);
                 if (!SCALAR) a4 = *reinterpret_cast<const float4*>(&a_s[t][lane * RC + i]);
                 const float qq[4] = {q4.x, q4.y, q4.z, q4.w}, kk[4] = {k4.x, k4.y, k4.z, k4.w}, aa[4] = {a4.x, a4.y, a4.z, a4.w};
@@ -430,7 +462,7 @@ __global__ void __launch_bounds__(THREADS) state_scan_wide_kernel(LinearStatePar
                 for (int u = 0; u < 4; u++)
 #pragma unroll
                     for (int c = 0; c < CW; c++) {
-                        st[i + u][c] = fmaf(aa[u], st[i + u][c], kk[u] * vv[c]);
+                        st[i + u][c] = WRITES ? fmaf(aa[u], vv[c] - st[i + u][c], st[i + u][c]) : fmaf(aa[u], st[i + u][c], kk[u] * vv[c]);
                         sum[c] = fmaf(st[i + u][c], qq[u], sum[c]);
                     }
             }
@@ -506,8 +538,9 @@ __global__ void __launch_bounds__(THREADS) state_scan_wide_kernel(LinearStatePar
 // owns 16 columns of one head's S; thread (group g of 8, column j of 16) takes the channels g, g + 8, ...
 // so that a warp's loads are whole 64-byte rows, keeps them in registers from load to store, and the
 // eight groups' sums meet in shared memory.  All state loads are issued before anything waits.
-template <typename T, int R, bool SCALAR>
+template <typename T, int R, int MODE>
 __global__ void __launch_bounds__(THREADS) state_step_kernel(LinearStateParams p) {
+    constexpr bool SCALAR = MODE == 1, WRITES = MODE == 2;
     __shared__ float q_s[SLICES * R], k_s[SLICES * R], a_s[SLICES * R];
     __shared__ float red[SLICES][COLS + 1];
     const int tid = threadIdx.x, jj = tid & (COLS - 1), g = tid >> 4;
@@ -539,6 +572,12 @@ __global__ void __launch_bounds__(THREADS) state_step_kernel(LinearStateParams p
     }
     for (int c = tid; c < SLICES * R; c += THREADS) {
         const bool there = c < d;
+        if (WRITES) {      // the gates of the one token are formed here: a step of single tokens runs no kernel ahead of this one
+            const int ch = h * d + c;
+            q_s[c] = there ? silu_f32(to_f32<T>(r[p.q_off + ch])) * p.q_scale : 0.f;
+            a_s[c] = there ? write_gate(p.decay[row * p.decay_stride + ch], p.gate_bias ? p.gate_bias[ch] : 0.f, p.lower[ch]) : 0.f;
+            continue;
+        }
         q_s[c] = there ? to_f32<T>(r[p.q_off + h * d + c]) * p.q_scale : 0.f;
         k_s[c] = there ? to_f32<T>(r[p.k_off + h * d + c]) * take : 0.f;
         a_s[c] = SCALAR ? keep : (there ? p.decay[row * p.decay_stride + h * d + c] : 1.f);
@@ -549,7 +588,7 @@ __global__ void __launch_bounds__(THREADS) state_step_kernel(LinearStateParams p
 #pragma unroll
     for (int i = 0; i < R; i++) {
         const int c = g + SLICES * i;
-        st[i] = fmaf(a_s[c], st[i], k_s[c] * vj);
+        st[i] = WRITES ? fmaf(a_s[c], vj - st[i], st[i]) : fmaf(a_s[c], st[i], k_s[c] * vj);
         acc = fmaf(st[i], q_s[c], acc);
     }
 #pragma unroll
@@ -576,43 +615,43 @@ __global__ void __launch_bounds__(THREADS) state_step_kernel(LinearStateParams p
     }
 }
 
-template <typename T, bool SCALAR>
+template <typename T, int MODE>
 int launch_step(const LinearStateParams& p, cudaStream_t stream) {
-    dim3 grid((p.dv + COLS - 1) / COLS + (SCALAR ? 1 : 0), p.heads, p.nseq);
+    dim3 grid((p.dv + COLS - 1) / COLS + (MODE == 1 ? 1 : 0), p.heads, p.nseq);
     if (grid.y > 65535 || grid.z > 65535) GB_REFUSE("state_scan: grid (%u, %u, %u) exceeds one launch", grid.x, grid.y, grid.z);
     if (p.d <= 64)
-        state_step_kernel<T, 8, SCALAR><<<grid, THREADS, 0, stream>>>(p);
+        state_step_kernel<T, 8, MODE><<<grid, THREADS, 0, stream>>>(p);
     else if (p.d <= 128)
-        state_step_kernel<T, 16, SCALAR><<<grid, THREADS, 0, stream>>>(p);
+        state_step_kernel<T, 16, MODE><<<grid, THREADS, 0, stream>>>(p);
     else
-        state_step_kernel<T, 32, SCALAR><<<grid, THREADS, 0, stream>>>(p);
+        state_step_kernel<T, 32, MODE><<<grid, THREADS, 0, stream>>>(p);
     GB_CHECK_LAUNCH("state_step");
     return 0;
 }
 
-template <typename T, bool SCALAR>
+template <typename T, int MODE>
 int launch_scan(const LinearStateParams& p, cudaStream_t stream) {
-    if (p.max_q_len == 1) return launch_step<T, SCALAR>(p, stream);   // every sequence brings one token
+    if (p.max_q_len == 1) return launch_step<T, MODE>(p, stream);   // every sequence brings one token
     const int rc = ((p.d + SLICES - 1) / SLICES + 3) / 4 * 4;
-    dim3 grid((p.dv + COLS - 1) / COLS + (SCALAR ? 1 : 0), p.heads, p.nseq);
+    dim3 grid((p.dv + COLS - 1) / COLS + (MODE == 1 ? 1 : 0), p.heads, p.nseq);
     if (grid.y > 65535 || grid.z > 65535) GB_REFUSE("state_scan: grid (%u, %u, %u) exceeds one launch", grid.x, grid.y, grid.z);
     if (p.d == 128 || p.d == 256) {     // heads whose channels fill a warp's 32 slices: shared memory read once
         if (p.d == 128)
-            state_scan_wide_kernel<T, 4, SCALAR><<<grid, THREADS, 0, stream>>>(p);
+            state_scan_wide_kernel<T, 4, MODE><<<grid, THREADS, 0, stream>>>(p);
         else
-            state_scan_wide_kernel<T, 8, SCALAR><<<grid, THREADS, 0, stream>>>(p);
+            state_scan_wide_kernel<T, 8, MODE><<<grid, THREADS, 0, stream>>>(p);
         GB_CHECK_LAUNCH("state_scan");
         return 0;
     }
     switch (rc) {
-        case 4: state_scan_kernel<T, 4, SCALAR><<<grid, THREADS, 0, stream>>>(p); break;
-        case 8: state_scan_kernel<T, 8, SCALAR><<<grid, THREADS, 0, stream>>>(p); break;
-        case 12: state_scan_kernel<T, 12, SCALAR><<<grid, THREADS, 0, stream>>>(p); break;
-        case 16: state_scan_kernel<T, 16, SCALAR><<<grid, THREADS, 0, stream>>>(p); break;
-        case 20: state_scan_kernel<T, 20, SCALAR><<<grid, THREADS, 0, stream>>>(p); break;
-        case 24: state_scan_kernel<T, 24, SCALAR><<<grid, THREADS, 0, stream>>>(p); break;
-        case 28: state_scan_kernel<T, 28, SCALAR><<<grid, THREADS, 0, stream>>>(p); break;
-        case 32: state_scan_kernel<T, 32, SCALAR><<<grid, THREADS, 0, stream>>>(p); break;
+        case 4: state_scan_kernel<T, 4, MODE><<<grid, THREADS, 0, stream>>>(p); break;
+        case 8: state_scan_kernel<T, 8, MODE><<<grid, THREADS, 0, stream>>>(p); break;
+        case 12: state_scan_kernel<T, 12, MODE><<<grid, THREADS, 0, stream>>>(p); break;
+        case 16: state_scan_kernel<T, 16, MODE><<<grid, THREADS, 0, stream>>>(p); break;
+        case 20: state_scan_kernel<T, 20, MODE><<<grid, THREADS, 0, stream>>>(p); break;
+        case 24: state_scan_kernel<T, 24, MODE><<<grid, THREADS, 0, stream>>>(p); break;
+        case 28: state_scan_kernel<T, 28, MODE><<<grid, THREADS, 0, stream>>>(p); break;
+        case 32: state_scan_kernel<T, 32, MODE><<<grid, THREADS, 0, stream>>>(p); break;
         default: GB_REFUSE("state_scan: %d key channels a head; at most 256", p.d);
     }
     GB_CHECK_LAUNCH("state_scan");
@@ -678,7 +717,7 @@ __global__ void __launch_bounds__(128) head_norm_gate_kernel(HeadGateParams p) {
             const int i = lane + 32 * e;
             const bool in = i < n;
             v[e] = in ? to_f32<TI>(x[i]) : 0.f;
-            z[e] = in ? to_f32<T>(g[i]) : 0.f;
+            z[e] = in && p.gate_kind != 2 ? to_f32<T>(g[i]) : 0.f;
             ww[e] = (in && w) ? w[i] : 1.f;
         }
 #pragma unroll
@@ -696,7 +735,7 @@ __global__ void __launch_bounds__(128) head_norm_gate_kernel(HeadGateParams p) {
             if (p.normed) o *= inv;
             if (w) o *= ww[e];
             const float sg = 1.f / (1.f + expf(-z[e]));
-            o *= p.gate_kind == 1 ? z[e] * sg : sg;
+            if (p.gate_kind != 2) o *= p.gate_kind == 1 ? z[e] * sg : sg;
             y[i] = from_f32<T>(o);
         }
         return;
@@ -715,9 +754,11 @@ __global__ void __launch_bounds__(128) head_norm_gate_kernel(HeadGateParams p) {
         if (p.divisor) v /= div;
         if (p.normed) v *= inv;
         if (w) v *= w[i];
-        const float z = to_f32<T>(g[i]);
-        const float s = 1.f / (1.f + expf(-z));
-        v *= p.gate_kind == 1 ? z * s : s;
+        if (p.gate_kind != 2) {
+            const float z = to_f32<T>(g[i]);
+            const float s = 1.f / (1.f + expf(-z));
+            v *= p.gate_kind == 1 ? z * s : s;
+        }
         y[i] = from_f32<T>(v);
     }
 }
@@ -745,7 +786,7 @@ __global__ void __launch_bounds__(128) head_norm_gate_span_kernel(HeadGateParams
         if (e < chunks) {
             const int i = 128 * e + 4 * lane;
             load4<TI>(x + i, v + 4 * e);
-            load4<T>(g + i, z + 4 * e);
+            if (p.gate_kind != 2) load4<T>(g + i, z + 4 * e);
             if (p.weight) {
                 const float* w = p.weight + (p.weight_per_head ? (int64_t)h0 * n + i : i % n);
                 const float4 w4 = *reinterpret_cast<const float4*>(w);
@@ -792,9 +833,9 @@ __global__ void __launch_bounds__(128) head_norm_gate_span_kernel(HeadGateParams
                 float t = v[4 * e + u];
                 if (p.normed) t *= inv[e];
                 if (p.weight) t *= ww[4 * e + u];
-                const float zz = z[4 * e + u];
+                const float zz = p.gate_kind == 2 ? 0.f : z[4 * e + u];
                 const float sg = 1.f / (1.f + expf(-zz));
-                o[u] = t * (p.gate_kind == 1 ? zz * sg : sg);
+                o[u] = p.gate_kind == 2 ? t : t * (p.gate_kind == 1 ? zz * sg : sg);
             }
             store4<T>(y + 128 * e + 4 * lane, o);
         }
@@ -841,12 +882,23 @@ GB_API int gb_state_scan(const LinearStateParams* pp, int dtype, cudaStream_t st
         if (p.head_stride < (int64_t)p.d * p.dv + p.d + 1) GB_REFUSE("state_scan: the state has no room for the normaliser and the maximum");
         mlstm_gates_kernel<<<dim3(p.heads, p.nseq), 32, 0, stream>>>(p);
         GB_CHECK_LAUNCH("mlstm_gates");
-        if (dtype == GB_F32) return launch_scan<float, true>(p, stream);
-        if (dtype == GB_BF16) return launch_scan<__nv_bfloat16, true>(p, stream);
+        if (dtype == GB_F32) return launch_scan<float, 1>(p, stream);
+        if (dtype == GB_BF16) return launch_scan<__nv_bfloat16, 1>(p, stream);
     } else {
         if (!p.decay) GB_REFUSE("state_scan: no decays");
-        if (dtype == GB_F32) return launch_scan<float, false>(p, stream);
-        if (dtype == GB_BF16) return launch_scan<__nv_bfloat16, false>(p, stream);
+        if (p.lower) {
+            if (dtype != GB_F32) GB_REFUSE("state_scan: rows whose forget gate writes are float32");
+            if (p.max_q_len != 1 && p.rows > 0) {
+                const int width = p.heads * p.d;
+                const int64_t total = (int64_t)p.rows * width;
+                forget_gate_kernel<<<(unsigned)((total + 255) / 256), 256, 0, stream>>>((float*)p.qkv + p.q_off, p.row_stride, (float*)p.decay,
+                                                                                       p.decay_stride, p.gate_bias, p.lower, total, width);
+                GB_CHECK_LAUNCH("forget_gate");
+            }
+            return launch_scan<float, 2>(p, stream);
+        }
+        if (dtype == GB_F32) return launch_scan<float, 0>(p, stream);
+        if (dtype == GB_BF16) return launch_scan<__nv_bfloat16, 0>(p, stream);
     }
     GB_REFUSE("state_scan: unknown dtype %d", dtype);
 }
@@ -855,7 +907,7 @@ GB_API int gb_head_norm_gate(const HeadGateParams* pp, int x_dtype, int dtype, c
     HeadGateParams p = *pp;
     if (p.rows <= 0) return 0;
     if (p.heads <= 0 || p.size <= 0) GB_REFUSE("head_norm_gate: %d heads of %d", p.heads, p.size);
-    if (p.gate_kind != 0 && p.gate_kind != 1) GB_REFUSE("head_norm_gate: gate kind %d", p.gate_kind);
+    if (p.gate_kind < 0 || p.gate_kind > 2 || (p.gate_kind == 2) != (p.gate == nullptr)) GB_REFUSE("head_norm_gate: gate kind %d", p.gate_kind);
     if (dtype == GB_F32 && x_dtype == GB_F32) return launch_gate<float, float>(p, stream);
     if (dtype == GB_BF16 && x_dtype == GB_F32) return launch_gate<float, __nv_bfloat16>(p, stream);
     if (dtype == GB_BF16 && x_dtype == GB_BF16) return launch_gate<__nv_bfloat16, __nv_bfloat16>(p, stream);

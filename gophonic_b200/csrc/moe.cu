@@ -6,6 +6,9 @@
 // products of a step of many rows multiply by, and as `top` (index, weight) pairs for a step of few rows
 // that reads only the chosen experts' matrices.
 //
+// With a correction an expert is chosen by its score plus a learned number and weighed by the score; with groups only
+// experts of the best groups of neighbours (by the sum of a group's two largest choice scores) can be chosen.
+//
 // moe_act: act[r, e * ff + i] = weight[r, e] * relu(up[r, e * ff + i])^2: the activation of every expert's
 // hidden layer with the row's weight for that expert folded in, so that one product with the experts' down
 // matrices side by side gives the weighted sum of the chosen experts' outputs (an expert that was not
@@ -28,7 +31,40 @@ namespace {
 
 constexpr int MAX_EXPERTS_PER_LANE = 16;   // experts up to 512
 
+// Which experts may be chosen: with groups, `key` (the warp's choice scores in shared memory) is scanned by a lane a group
+// for the group's two largest, and a group is kept if fewer than keep_groups groups come before it (a larger sum, or an
+// equal one and a lower number).  Scores of the other groups become -inf.
+__device__ __forceinline__ void drop_groups(float* key, float* strength, int E, int groups, int keep, int lane) {
+    const int per = E / groups;
+    for (int g = lane; g < groups; g += 32) {
+        float a = -INFINITY, b = -INFINITY;
+        for (int i = 0; i < per; i++) {
+            const float v = key[g * per + i];
+            if (v > a) {
+                b = a;
+                a = v;
+            } else if (v > b) {
+                b = v;
+            }
+        }
+        strength[g] = per > 1 ? a + b : a;
+    }
+    __syncwarp();
+    for (int g = lane; g < groups; g += 32) {
+        const float mine = strength[g];
+        int before = 0;
+        for (int o = 0; o < groups; o++) before += strength[o] > mine || (strength[o] == mine && o < g);
+        if (before >= keep)
+            for (int i = 0; i < per; i++) key[g * per + i] = -INFINITY;
+    }
+    __syncwarp();
+}
+
+// CORRECTED: the choice goes by score + correction and, with groups, inside the best of them
+template <bool CORRECTED>
 __global__ void __launch_bounds__(128) moe_route_kernel(MoeRouteParams p) {
+    __shared__ float key_s[CORRECTED ? 4 : 1][CORRECTED ? 32 * MAX_EXPERTS_PER_LANE : 1];
+    __shared__ float group_s[CORRECTED ? 4 : 1][CORRECTED ? 32 * MAX_EXPERTS_PER_LANE : 1];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int64_t row = (int64_t)blockIdx.x * 4 + warp;
     if (row >= p.rows) return;
@@ -55,6 +91,22 @@ __global__ void __launch_bounds__(128) moe_route_kernel(MoeRouteParams p) {
     }
     sum = warp_sum(sum);
     const float inv = p.score_kind == 1 ? 1.f : 1.f / sum;     // a sigmoid score stands by itself
+    if (CORRECTED) {
+#pragma unroll
+        for (int e = 0; e < MAX_EXPERTS_PER_LANE; e++) {
+            const int i = lane + 32 * e;
+            if (i >= E) continue;
+            s[e] = (p.score_kind == 1 ? 1.f / (1.f + expf(-s[e])) : s[e] * inv) + (p.correction ? p.correction[i] : 0.f);
+            if (p.groups > 1) key_s[warp][i] = s[e];
+        }
+        if (p.groups > 1) {
+            __syncwarp();
+            drop_groups(key_s[warp], group_s[warp], E, p.groups, p.keep_groups, lane);
+#pragma unroll
+            for (int e = 0; e < MAX_EXPERTS_PER_LANE; e++)
+                if (lane + 32 * e < E) s[e] = key_s[warp][lane + 32 * e];
+        }
+    }
     float* dense = p.dense + row * E;
     for (int i = lane; i < E; i += 32) dense[i] = 0.f;
     float chosen_sum = 0.f;
@@ -77,7 +129,14 @@ __global__ void __launch_bounds__(128) moe_route_kernel(MoeRouteParams p) {
 #pragma unroll
         for (int e = 0; e < MAX_EXPERTS_PER_LANE; e++)
             if (lane + 32 * e == best_i) s[e] = -INFINITY;
-        const float sc = p.score_kind == 1 ? 1.f / (1.f + expf(-best)) : best * inv;
+        if (best_i >= E) best_i = k;       // no number compares (NaN logits): any expert, but one that exists
+        float sc;
+        if (CORRECTED) {       // the score again, without its correction
+            const float zc = z[best_i];
+            sc = p.score_kind == 1 ? 1.f / (1.f + expf(-zc)) : expf(zc - mx) * inv;
+        } else {
+            sc = p.score_kind == 1 ? 1.f / (1.f + expf(-best)) : best * inv;
+        }
         chosen_sum += sc;
         if (lane == (k & 31)) my_w = sc, my_i = best_i;
         if (k >= 32 && lane == 0) {}   // more than 32 choices are refused on the host
@@ -358,7 +417,12 @@ GB_API int gb_moe_route(const MoeRouteParams* pp, cudaStream_t stream) {
     if (p.experts <= 0 || p.experts > 32 * MAX_EXPERTS_PER_LANE) GB_REFUSE("moe_route: %d experts; 1 to %d", p.experts, 32 * MAX_EXPERTS_PER_LANE);
     if (p.top <= 0 || p.top > p.experts || p.top > 32) GB_REFUSE("moe_route: %d of %d experts a token; at most 32", p.top, p.experts);
     if (!p.logits || !p.dense || !p.index || !p.weight) GB_REFUSE("moe_route: a tensor is missing");
-    moe_route_kernel<<<(p.rows + 3) / 4, 128, 0, stream>>>(p);
+    if (p.groups > 1 && (p.experts % p.groups || p.keep_groups <= 0 || p.keep_groups > p.groups || p.experts / p.groups * p.keep_groups < p.top))
+        GB_REFUSE("moe_route: %d of %d experts a token out of the best %d of %d groups", p.top, p.experts, p.keep_groups, p.groups);
+    if (p.correction || p.groups > 1)
+        moe_route_kernel<true><<<(p.rows + 3) / 4, 128, 0, stream>>>(p);
+    else
+        moe_route_kernel<false><<<(p.rows + 3) / 4, 128, 0, stream>>>(p);
     GB_CHECK_LAUNCH("moe_route");
     return 0;
 }

@@ -58,11 +58,15 @@ class Model:
         self.streams = int(getattr(spec, "streams", 1))
         if any(self._takes_streams) != all(self._takes_streams) or (self.streams > 1 and not all(self._takes_streams)):
             raise ValueError("model spec: a residual kept in streams needs blocks that take streams, all of them")
+        # ... or it may read the results of all earlier layer runs; then every block must take them as planes
+        self._takes_history = [bool(getattr(b, "takes_history", False)) for b in self.blocks]
+        if any(self._takes_history) and (not all(self._takes_history) or any(self._takes_streams)):
+            raise ValueError("model spec: blocks that read earlier layers' results stand only beside blocks of their kind")
         # junctions: parts that rewrite the residual right before a run of the schedule
         self.junctions = {pos: registry.part_class("junction", e.enter.kind)(e.enter, "", tensors, runtime)
                           for pos, e in enumerate(spec.schedule) if getattr(e, "enter", None) is not None}
-        if self.junctions and self._takes_streams[0]:
-            raise ValueError("model spec: a junction rewrites one residual; blocks that keep it in streams cannot have one")
+        if self.junctions and (self._takes_streams[0] or self._takes_history[0]):
+            raise ValueError("model spec: a junction rewrites one residual; blocks that keep it in streams or planes cannot have one")
         # a block arrangement may take the norm that follows it (to prepare the residual's rows for it)
         self._takes_next_norm = ["next_norm" in inspect.signature(b.forward).parameters for b in self.blocks]
         norm_prefix = final_norm_prefix(spec)
@@ -149,6 +153,8 @@ class Model:
         rows = batch.rows
         if self._takes_streams[0]:
             return self._forward_streams(batch, cache, want_rows)
+        if self._takes_history[0]:
+            return self._forward_history(batch, cache, want_rows)
         h = torch.empty((rows, self.spec.hidden), dtype=torch.float32, device=self.rt.device)
         # What is still owed to the residual travels from block to block: an addend not yet added, the
         # rows' statistics (``RowStats``) where the last kernel left them, or nothing.
@@ -193,9 +199,33 @@ class Model:
         n = want_rows.numel()
         x = torch.empty((n, self.spec.hidden), dtype=self.rt.act_dtype, device=self.rt.device)
         self.final_norm.forward(h, x, delta, rows=want_rows)
-        logits = torch.empty((n, self.spec.vocab), dtype=torch.float32, device=self.rt.device)
+        return self._logits(x)
+
+    def _logits(self, x: torch.Tensor) -> torch.Tensor:
+        """The head's float32 logits of normed rows."""
+        ops = self.rt.ops
+        logits = torch.empty((x.shape[0], self.spec.vocab), dtype=torch.float32, device=self.rt.device)
         ops.gemm(x, self.head, logits)
+        cap = float(getattr(self.spec.head, "soft_cap", 0.0))
+        if cap > 0.0:
+            ops.soft_cap_(logits, cap)
         return logits
+
+    def _forward_history(self, batch, cache: Cache, want_rows: Optional[torch.Tensor]) -> Optional[torch.Tensor]:
+        """The same pass for blocks that read the results of all earlier runs: plane 0 of the results is the embedding
+        output, run i leaves plane i + 1, and what the last block leaves unfinished is completed for the wanted rows alone."""
+        ops = self.rt.ops
+        schedule = self.spec.schedule
+        planes = torch.empty((len(schedule) + 1, batch.rows, self.spec.hidden), dtype=torch.float32, device=self.rt.device)
+        ops.embed_gather(self.embedding, batch.ids, planes[0], scale=float(getattr(self.spec.embedding, "scale", 1.0)))
+        pending = None
+        for pos, entry in enumerate(schedule):
+            pending = self.blocks[entry.layer].forward(batch, planes, pos, pending, cache.view(pos))
+        if want_rows is None or want_rows.numel() == 0:
+            return None
+        x = torch.empty((want_rows.numel(), self.spec.hidden), dtype=self.rt.act_dtype, device=self.rt.device)
+        self.blocks[schedule[-1].layer].finish(planes, pending, self.final_norm, x, want_rows)
+        return self._logits(x)
 
     def _forward_streams(self, batch, cache: Cache, want_rows: Optional[torch.Tensor]) -> Optional[torch.Tensor]:
         """The same pass for blocks that keep the residual in streams: all streams start as the embedding
@@ -214,6 +244,4 @@ class Model:
         n = want_rows.numel()
         x = torch.empty((n, self.spec.hidden), dtype=self.rt.act_dtype, device=self.rt.device)
         self.blocks[self.spec.schedule[-1].layer].finish(streams, pending, self.final_norm, x, want_rows)
-        logits = torch.empty((n, self.spec.vocab), dtype=torch.float32, device=self.rt.device)
-        ops.gemm(x, self.head, logits)
-        return logits
+        return self._logits(x)

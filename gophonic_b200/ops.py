@@ -521,7 +521,7 @@ def checked_status():
     found out of bounds since the last call (the access was skipped or redirected, nothing faulted).
     Always None in the ordinary build, whose kernels carry no checks.  Synchronises."""
     out = (c_int * 4)()
-    for name in ("rows", "cache", "attention_simt", "attention_mma", "attention_tc5", "linear_state", "delta_state", "attention_sigmoid", "hyper", "postnorm", "attention_latent"):
+    for name in ("rows", "cache", "attention_simt", "attention_mma", "attention_tc5", "linear_state", "delta_state", "attention_sigmoid", "hyper", "postnorm", "attention_latent", "sandwich"):
         code = int(getattr(_lib, "gb_checked_status_" + name)(out))
         if code or out[3]:
             return name, _CHECK_NAMES.get(code, f"code {code}"), out[1], out[2], out[3]
@@ -546,6 +546,7 @@ class _QkRopeParams(Structure):
         ("write_kv", c_int), ("rows", c_int), ("heads", c_int), ("kv_heads", c_int), ("d", c_int),
         ("pages", c_int), ("max_slots", c_int),
         ("q_b", c_void_p), ("k_b", c_void_p), ("v_b", c_void_p), ("pairs", c_int), ("dv", c_int), ("span", c_int), ("v_share", c_int),
+        ("v_from_k", c_int),
     ]
 
 
@@ -555,12 +556,14 @@ def _rope_params(qkv: torch.Tensor, heads: int, kv_heads: int, head_dim: int,
                  row_pos: torch.Tensor, row_seq: torch.Tensor, seq_slot: torch.Tensor,
                  block_table: torch.Tensor,
                  k_plane: Optional[torch.Tensor], v_plane: Optional[torch.Tensor], write_kv: bool,
-                 biases=None, pairs: bool = False, value_dim: Optional[int] = None, span: bool = False, v_share: int = 1) -> "_QkRopeParams":
+                 biases=None, pairs: bool = False, value_dim: Optional[int] = None, span: bool = False, v_share: int = 1,
+                 value_from_key: bool = False) -> "_QkRopeParams":
     """``biases`` = (q, k, v) float32 vectors or None each, added to the heads first; ``pairs``: channels
     2j and 2j + 1 turn together instead of j and j + rotary_dim / 2; ``value_dim``: size of a value
     head if it is not ``head_dim``; ``span``: the norm runs over all heads of q together (``q_weight`` of
     heads * head_dim) and over all heads of k together, not per head; ``v_share`` > 1: that many consecutive
-    key heads read one value head, so the row and the value plane hold kv_heads / v_share value heads.  With any
+    key heads read one value head, so the row and the value plane hold kv_heads / v_share value heads;
+    ``value_from_key``: the row holds no value heads, a value is its key as it stands in the row, before norm and rotation.  With any
     of them the rows may be wider than q, k and v (what follows them is left alone)."""
     _need(qkv, "qkv", dim=2, contiguous=False)
     rows = qkv.shape[0]
@@ -569,8 +572,10 @@ def _rope_params(qkv: torch.Tensor, heads: int, kv_heads: int, head_dim: int,
     if kv_heads % v_share:
         raise KernelError(f"qk_norm_rope: {kv_heads} key heads share value heads by {v_share}")
     v_heads = kv_heads // v_share
-    general = biases is not None or pairs or dv != head_dim or span or v_share > 1
-    used = (heads + kv_heads) * head_dim + v_heads * dv
+    if value_from_key and (v_share > 1 or dv != head_dim or biases is not None):
+        raise KernelError("qk_norm_rope: values that are the keys are as many and as wide as the keys and have no biases")
+    general = biases is not None or pairs or dv != head_dim or span or v_share > 1 or value_from_key
+    used = (heads + kv_heads) * head_dim + (0 if value_from_key else v_heads * dv)
     if qkv.stride(1) != 1 or (qkv.shape[1] < used if general else (qkv.shape[1] != used or not qkv.is_contiguous())):
         raise KernelError(f"qk_norm_rope: qkv {tuple(qkv.shape)} for {heads}+{kv_heads} heads of {head_dim} and {kv_heads} of {dv}")
     q_b, k_b, v_b = biases if biases is not None else (None, None, None)
@@ -608,7 +613,8 @@ def _rope_params(qkv: torch.Tensor, heads: int, kv_heads: int, head_dim: int,
                       1 if write_kv else 0, rows, heads, kv_heads, head_dim,
                       0 if k_plane is None else k_plane.shape[0], block_table.shape[0],
                       0 if q_b is None else q_b.data_ptr(), 0 if k_b is None else k_b.data_ptr(),
-                      0 if v_b is None else v_b.data_ptr(), 1 if pairs else 0, dv, 1 if span else 0, v_share)
+                      0 if v_b is None else v_b.data_ptr(), 1 if pairs else 0, dv, 1 if span else 0, v_share,
+                      1 if value_from_key else 0)
     return p
 
 
@@ -747,7 +753,7 @@ class _LinearStateParams(Structure):
         ("gate_cap", c_float), ("coef", c_void_p), ("state", c_void_p), ("slot_stride", c_int64), ("head_stride", c_int64),
         ("out", c_void_p), ("out_stride", c_int64), ("seq_slot", c_void_p), ("seq_q_start", c_void_p), ("seq_q_len", c_void_p),
         ("nseq", c_int), ("heads", c_int), ("d", c_int), ("dv", c_int), ("scalar_decay", c_int), ("max_slots", c_int),
-        ("max_q_len", c_int),
+        ("max_q_len", c_int), ("lower", c_void_p), ("rows", c_int),
     ]
 
 
@@ -759,7 +765,7 @@ class _HeadGateParams(Structure):
     ]
 
 
-GATE_SIGMOID, GATE_SILU = 0, 1
+GATE_SIGMOID, GATE_SILU, GATE_NONE = 0, 1, 2
 
 
 def gla_decay(z: torch.Tensor, bias: Optional[torch.Tensor], tau: float) -> None:
@@ -776,7 +782,7 @@ def state_scan(qkv: torch.Tensor, q_off: int, k_off: int, v_off: int, heads: int
                state: torch.Tensor, out: torch.Tensor, seq_slot: torch.Tensor, seq_q_start: torch.Tensor, seq_q_len: torch.Tensor,
                nseq: int, decay: Optional[torch.Tensor] = None, gates: Optional[torch.Tensor] = None,
                gate_bias: Optional[torch.Tensor] = None, gate_cap: float = 0.0, coef: Optional[torch.Tensor] = None,
-               max_q_len: int = 0) -> None:
+               max_q_len: int = 0, lower: Optional[torch.Tensor] = None) -> None:
     """The matrix-state recurrence S <- diag(a) S + b k v^T, o = S^T (q * q_scale) over the rows of a step,
     token by token, for every (sequence, head); ``state`` [slots, heads, d * dv (+ d + 1)] float32 is read
     and left updated, ``out`` [rows, heads * dv] float32 receives the sums.  With ``decay`` (float32 [rows,
@@ -785,7 +791,12 @@ def state_scan(qkv: torch.Tensor, q_off: int, k_off: int, v_off: int, heads: int
     a and b are the stabilised exponential gates of a matrix memory, the state also carries the
     normaliser and the running maximum, and coef[..., 3] receives each token's divisor.  ``max_q_len``:
     the most rows a sequence brings, if known (1: every sequence brings one token, which has a kernel
-    of its own; the arithmetic per element is the same)."""
+    of its own; the arithmetic per element is the same).
+
+    With ``lower`` (float32 [heads * d]) the forget gate also decides what is written: ``decay`` then holds its
+    pre-activations z (in the rows of ``qkv`` or anywhere), ``gate_bias`` [heads * d] is added to them, and with
+    u = (1 - lower) sigmoid(-z) the state goes S <- S + u (v - S) (there is no key: ``k_off`` is ignored) and o = S^T silu(q).
+    ``qkv`` is float32 and a step of more than one token a sequence overwrites q and z by silu(q) and u."""
     _need(qkv, "state_scan rows", dim=2, contiguous=False)
     _need(state, "state", torch.float32, 3)
     _need(out, "state_scan out", torch.float32, 2)
@@ -805,6 +816,8 @@ def state_scan(qkv: torch.Tensor, q_off: int, k_off: int, v_off: int, heads: int
         _need(coef, "gate factors", torch.float32, 3)
         if gates.shape != (rows, 2 * heads) or gates.stride(1) != 1 or coef.shape[0] < rows or coef.shape[1:] != (heads, 4):
             raise KernelError(f"state_scan: gates {tuple(gates.shape)}, factors {tuple(coef.shape)}")
+        if lower is not None:
+            raise KernelError("state_scan: lower bounds go with decays, not with gates")
         if gate_bias is not None:
             _need(gate_bias, "gate bias", torch.float32, 1)
             if gate_bias.numel() != 2 * heads:
@@ -815,30 +828,45 @@ def state_scan(qkv: torch.Tensor, q_off: int, k_off: int, v_off: int, heads: int
         _need(decay, "decays", torch.float32, 2, contiguous=False)
         if decay.shape != (rows, heads * d) or decay.stride(1) != 1:
             raise KernelError(f"state_scan: decays {tuple(decay.shape)} for {heads} heads of {d}")
+        if lower is not None:
+            for t, nm in ((lower, "lower bounds"), (gate_bias, "gate bias")):
+                if t is None:
+                    continue
+                _need(t, nm, torch.float32, 1)
+                if t.numel() != heads * d:
+                    raise KernelError(f"state_scan: {nm} of {t.numel()} for {heads} heads of {d}")
+            if qkv.dtype != torch.float32:
+                raise KernelError("state_scan: rows with lower bounds are float32")
+            k_off = q_off
     p = _LinearStateParams(qkv.data_ptr(), qkv.stride(0), q_off, k_off, v_off, q_scale,
                            0 if decay is None else decay.data_ptr(), 0 if decay is None else decay.stride(0),
                            0 if gates is None else gates.data_ptr(), 0 if gates is None else gates.stride(0),
                            0 if gate_bias is None else gate_bias.data_ptr(), gate_cap, 0 if coef is None else coef.data_ptr(),
                            state.data_ptr(), state.stride(0), state.stride(1), out.data_ptr(), out.stride(0),
                            seq_slot.data_ptr(), seq_q_start.data_ptr(), seq_q_len.data_ptr(), nseq, heads, d, dv,
-                           1 if scalar else 0, state.shape[0], int(max_q_len))
-    _check(_lib.gb_state_scan(byref(p), _code(qkv.dtype), _stream()), 2 if scalar else 1)
+                           1 if scalar else 0, state.shape[0], int(max_q_len), 0 if lower is None else lower.data_ptr(), rows)
+    _check(_lib.gb_state_scan(byref(p), _code(qkv.dtype), _stream()), 2 if scalar or (lower is not None and max_q_len != 1) else 1)
 
 
-def head_norm_gate(x: torch.Tensor, gate: torch.Tensor, y: torch.Tensor, heads: int, size: int, gate_kind: int,
+def head_norm_gate(x: torch.Tensor, gate: Optional[torch.Tensor], y: torch.Tensor, heads: int, size: int, gate_kind: int,
                    weight: Optional[torch.Tensor] = None, eps: Optional[float] = None, divisor: Optional[torch.Tensor] = None) -> None:
     """y[r, h] = norm(x[r, h] / divisor[r, h]) * weight * gate(g[r, h]) for heads of ``size``: the division
     only with ``divisor`` (float32 [rows, heads, 1], possibly a column of a wider tensor), the norm (x over its root mean
     square, eps under the root) only with ``eps``, the weight ([size], shared by the heads, or
-    [heads * size]) only if given; the gate is sigmoid(g) or, with ``GATE_SILU``, g * sigmoid(g).
+    [heads * size]) only if given; the gate is sigmoid(g) or, with ``GATE_SILU``, g * sigmoid(g), or there is none
+    (``GATE_NONE``, ``gate`` None).
     x is float32 or the activation dtype; g and y are the activation dtype; all arithmetic float32."""
     _need(x, "head_norm_gate x", dim=2, contiguous=False)
-    _need(gate, "head_norm_gate gate", y.dtype, 2, contiguous=False)
+    if (gate is None) != (gate_kind == GATE_NONE):
+        raise KernelError("head_norm_gate: a gate and a kind of gate go together")
+    if gate is not None:
+        _need(gate, "head_norm_gate gate", y.dtype, 2, contiguous=False)
     _need(y, "head_norm_gate y", dim=2, contiguous=False)
     rows = x.shape[0]
     n = heads * size
-    if (x.shape[1] < n or gate.shape != (rows, n) or y.shape != (rows, n) or x.stride(1) != 1 or gate.stride(1) != 1 or y.stride(1) != 1):
-        raise KernelError(f"head_norm_gate: x {tuple(x.shape)}, gate {tuple(gate.shape)}, y {tuple(y.shape)} for {heads} heads of {size}")
+    if (x.shape[1] < n or y.shape != (rows, n) or x.stride(1) != 1 or y.stride(1) != 1
+            or (gate is not None and (gate.shape != (rows, n) or gate.stride(1) != 1))):
+        raise KernelError(f"head_norm_gate: x {tuple(x.shape)}, gate {None if gate is None else tuple(gate.shape)}, y {tuple(y.shape)} for {heads} heads of {size}")
     per_head = 0
     if weight is not None:
         _need(weight, "head norm weight", torch.float32, 1)
@@ -851,7 +879,7 @@ def head_norm_gate(x: torch.Tensor, gate: torch.Tensor, y: torch.Tensor, heads: 
         dstride = divisor.stride(1)
         if divisor.shape[0] < rows or divisor.shape[1] != heads or divisor.stride(0) != heads * dstride:
             raise KernelError(f"head_norm_gate: divisor {tuple(divisor.shape)} with strides {divisor.stride()}")
-    p = _HeadGateParams(x.data_ptr(), x.stride(0), gate.data_ptr(), gate.stride(0), y.data_ptr(), y.stride(0),
+    p = _HeadGateParams(x.data_ptr(), x.stride(0), 0 if gate is None else gate.data_ptr(), 0 if gate is None else gate.stride(0), y.data_ptr(), y.stride(0),
                         0 if divisor is None else divisor.data_ptr(), dstride, 0 if weight is None else weight.data_ptr(), per_head,
                         0 if eps is None else 1, 0.0 if eps is None else eps, gate_kind, rows, heads, size)
     _check(_lib.gb_head_norm_gate(byref(p), _code(x.dtype), _code(y.dtype), _stream()))
@@ -1253,7 +1281,8 @@ def attention_sigmoid(q: torch.Tensor, out: torch.Tensor, k_plane: torch.Tensor,
 # ---- mixture of experts -----------------------------------------------------------------------
 class _MoeRouteParams(Structure):
     _fields_ = [("logits", c_void_p), ("logits_stride", c_int64), ("rows", c_int), ("experts", c_int), ("top", c_int),
-                ("renorm_eps", c_float), ("dense", c_void_p), ("index", c_void_p), ("weight", c_void_p), ("score_kind", c_int), ("renorm", c_int)]
+                ("renorm_eps", c_float), ("dense", c_void_p), ("index", c_void_p), ("weight", c_void_p), ("score_kind", c_int), ("renorm", c_int),
+                ("correction", c_void_p), ("groups", c_int), ("keep_groups", c_int)]
 
 
 class _MoeRowsParams(Structure):
@@ -1267,11 +1296,15 @@ MOE_ACTS = {"relu2": 0, "swiglu": 1, "glu_clamp": 2}     # the last two are gate
 
 
 def moe_route(logits: torch.Tensor, top: int, renorm_eps: float, dense: torch.Tensor, index: torch.Tensor, weight: torch.Tensor,
-              score: str = "softmax", renorm: bool = True) -> None:
+              score: str = "softmax", renorm: bool = True, correction: Optional[torch.Tensor] = None, groups: int = 1,
+              keep_groups: int = 1) -> None:
     """Per row of ``logits`` (float32 [rows, experts]): scores (softmax over the experts, or with ``score``
     "sigmoid" the sigmoid of each logit by itself), the ``top`` largest chosen, their weights s / (sum of the
     chosen + renorm_eps), or with ``renorm`` False the scores themselves, left in ``dense`` (float32 [rows,
-    experts], zeros elsewhere) and as pairs in ``index`` (int32 [rows, top]) and ``weight`` (float32 [rows, top])."""
+    experts], zeros elsewhere) and as pairs in ``index`` (int32 [rows, top]) and ``weight`` (float32 [rows, top]).
+    ``correction`` (float32 [experts]): an expert is chosen by its score plus this number, its weight comes from the score.
+    ``groups`` > 1: the experts form that many equal groups of neighbours and only experts of the ``keep_groups`` groups
+    whose two largest choice scores add up to most (the lower group first of equal ones) can be chosen."""
     _need(logits, "router logits", torch.float32, 2, contiguous=False)
     rows, experts = logits.shape
     _need(dense, "expert weights", torch.float32, 2)
@@ -1279,8 +1312,12 @@ def moe_route(logits: torch.Tensor, top: int, renorm_eps: float, dense: torch.Te
     _need(weight, "chosen weights", torch.float32, 2)
     if logits.stride(1) != 1 or dense.shape != (rows, experts) or index.shape != (rows, top) or weight.shape != (rows, top):
         raise KernelError(f"moe_route: logits {tuple(logits.shape)}, dense {tuple(dense.shape)}, pairs {tuple(index.shape)} / {tuple(weight.shape)}")
+    if correction is not None:
+        _need(correction, "choice correction", torch.float32, 1)
+        if correction.numel() != experts:
+            raise KernelError(f"moe_route: {correction.numel()} corrections for {experts} experts")
     p = _MoeRouteParams(logits.data_ptr(), logits.stride(0), rows, experts, top, renorm_eps, dense.data_ptr(), index.data_ptr(), weight.data_ptr(),
-                        MOE_SCORES[score], 1 if renorm else 0)
+                        MOE_SCORES[score], 1 if renorm else 0, 0 if correction is None else correction.data_ptr(), int(groups), int(keep_groups))
     _check(_lib.gb_moe_route(byref(p), _stream()))
 
 
@@ -1623,3 +1660,105 @@ def head_gemm_mma(a: torch.Tensor, w_nk: torch.Tensor, out: torch.Tensor) -> Non
         raise KernelError(f"head_gemm_mma: a {tuple(a.shape)}, w {tuple(w_nk.shape)}, out {tuple(out.shape)}")
     _check(_lib.gb_head_gemm_mma(_ptr(a), c_int64(a.stride(0)), c_int64(a.stride(1)), _ptr(w_nk), _ptr(out), c_int64(out.stride(0)),
                                  c_int64(out.stride(1)), c_int(rows), c_int(heads), c_int(K), c_int(N), _stream()))
+
+
+# ---- blocks with norms on both sides, a short convolution and a weighted sum over the depth -----------------
+class _SandwichParams(Structure):
+    _fields_ = [
+        ("base", c_void_p), ("y", c_void_p), ("y_w", c_void_p), ("y_eps", c_float), ("result", c_void_p),
+        ("planes", c_void_p), ("plane_stride", c_int64), ("n_planes", c_int), ("average", c_void_p), ("x_out", c_void_p),
+        ("norm_w", c_void_p), ("norm_eps", c_float), ("out", c_void_p), ("row_index", c_void_p),
+        ("conv_w", c_void_p), ("taps", c_int), ("state", c_void_p), ("state_slot_stride", c_int64), ("row_seq", c_void_p),
+        ("seq_slot", c_void_p), ("max_slots", c_int), ("rows", c_int), ("width", c_int),
+    ]
+
+
+def _conv_state(conv: torch.Tensor, state: Optional[torch.Tensor], width: int, who: str):
+    _need(conv, "convolution weights", torch.float32, 2)
+    taps = conv.shape[0]
+    if conv.shape[1] != width:
+        raise KernelError(f"{who}: convolution weights {tuple(conv.shape)} for rows of {width}")
+    if taps > 1:
+        if state is None:
+            raise KernelError(f"{who}: a convolution needs the sequences' state")
+        _need(state, "convolution state", torch.float32, 2, contiguous=False)
+        if state.shape[1] < (taps - 1) * width or state.stride(1) != 1:
+            raise KernelError(f"{who}: state {tuple(state.shape)} for {taps - 1} rows of {width}")
+    return taps
+
+
+def sandwich_rows(base: torch.Tensor, out: torch.Tensor, norm_weight: torch.Tensor, eps: float, y: Optional[torch.Tensor] = None,
+                  y_weight: Optional[torch.Tensor] = None, y_eps: float = 0.0, result: Optional[torch.Tensor] = None,
+                  planes: Optional[torch.Tensor] = None, n_planes: int = 0, average: Optional[torch.Tensor] = None,
+                  x_out: Optional[torch.Tensor] = None, rows: Optional[torch.Tensor] = None, conv: Optional[torch.Tensor] = None,
+                  state: Optional[torch.Tensor] = None, batch=None) -> None:
+    """One pass over rows of the residual (float32 [rows, width]) between two sublayers:
+
+        v = base + y / sqrt(mean(y^2) + y_eps) * y_weight          (no ``y``: v = base)      -> ``result`` if given
+        x = sum over j < n_planes of average[j] planes[j] + average[n_planes] v   (no ``average``: x = v)   -> ``x_out`` if given
+        out = x / sqrt(mean(x^2) + eps) * norm_weight              float32 or bfloat16
+
+    With ``conv`` (float32 [taps, width]; every row is then the single token of its sequence) the normed row h is convolved
+    over time on its way out, out = h + sum_j conv[j] h_(t - taps + 1 + j), the earlier rows coming from ``state``
+    (float32 [slots, (taps - 1) * width], oldest first), which is moved on by this token.  With ``rows`` (int32 indices)
+    out[i] is made from row rows[i] and nothing but ``out`` is written."""
+    _need(base, "residual", torch.float32, 2)
+    _need(out, "normed rows", dim=2)
+    n, width = base.shape
+    out_rows = n
+    if rows is not None:
+        _need(rows, "row index", torch.int32, 1)
+        out_rows = rows.numel()
+        if result is not None or x_out is not None or conv is not None:
+            raise KernelError("sandwich_rows: gathered rows leave everything but the normed rows as it is")
+    if out.shape != (out_rows, width):
+        raise KernelError(f"sandwich_rows: normed rows {tuple(out.shape)}, want {(out_rows, width)}")
+    for t, nm, shape in ((y, "sublayer output", (n, width)), (result, "result", (n, width)), (x_out, "averaged rows", (n, width)),
+                         (norm_weight, "norm weight", (width,)), (y_weight, "output norm weight", (width,))):
+        if t is not None:
+            _need(t, nm, torch.float32)
+            if tuple(t.shape) != shape:
+                raise KernelError(f"sandwich_rows: {nm} {tuple(t.shape)}, want {shape}")
+    if (y is None) != (y_weight is None):
+        raise KernelError("sandwich_rows: a sublayer's output and its norm's weight go together")
+    if average is not None:
+        _need(planes, "result planes", torch.float32, 3)
+        _need(average, "average weights", torch.float32, 1)
+        if tuple(planes.shape[1:]) != (n, width) or not 0 <= n_planes <= planes.shape[0] or average.numel() != n_planes + 1:
+            raise KernelError(f"sandwich_rows: {average.numel()} weights for {n_planes} planes of {tuple(planes.shape)} and one row more")
+    taps = 0
+    if conv is not None:
+        taps = _conv_state(conv, state, width, "sandwich_rows")
+        if batch is None or batch.max_q_len != 1 or batch.nseq != n:
+            raise KernelError("sandwich_rows: the convolution inside takes steps of single tokens")
+    p = _SandwichParams(base.data_ptr(), 0 if y is None else y.data_ptr(), 0 if y_weight is None else y_weight.data_ptr(), y_eps,
+                        0 if result is None else result.data_ptr(), 0 if average is None else planes.data_ptr(),
+                        0 if average is None else planes.stride(0), int(n_planes), 0 if average is None else average.data_ptr(),
+                        0 if x_out is None else x_out.data_ptr(), norm_weight.data_ptr(), eps, out.data_ptr(),
+                        0 if rows is None else rows.data_ptr(), 0 if conv is None else conv.data_ptr(), taps,
+                        0 if taps <= 1 else state.data_ptr(), 0 if taps <= 1 else state.stride(0),
+                        0 if conv is None else batch.row_seq.data_ptr(), 0 if conv is None else batch.seq_slot.data_ptr(),
+                        0 if taps <= 1 else state.shape[0], out_rows, width)
+    _check(_lib.gb_sandwich_rows(byref(p), _code(out.dtype), _stream()))
+
+
+def conv_rows(h: torch.Tensor, conv: torch.Tensor, state: Optional[torch.Tensor], out: torch.Tensor, batch) -> None:
+    """out[t] = h[t] + sum_j conv[j] h[t - taps + 1 + j] on every channel of the packed rows ``h`` (float32 [rows, width];
+    ``conv`` float32 [taps, width]): a tap reaches back into the step's earlier rows of the same sequence and, before them,
+    into ``state`` (float32 [slots, (taps - 1) * width], the sequence's last rows, oldest first), which is left updated."""
+    _need(h, "rows", torch.float32, 2)
+    _need(out, "convolved rows", dim=2)
+    rows, width = h.shape
+    if out.shape != h.shape:
+        raise KernelError(f"conv_rows: rows {tuple(h.shape)}, out {tuple(out.shape)}")
+    taps = _conv_state(conv, state, width, "conv_rows")
+    _check(_lib.gb_conv_rows(_ptr(h), _ptr(conv), c_int(taps), _ptr(state if taps > 1 else None), c_int64(state.stride(0) if taps > 1 else 0),
+                             c_int(state.shape[0] if taps > 1 else 0), _ptr(out), _code(out.dtype), c_int(rows), c_int(width), c_int(batch.nseq),
+                             _ptr(batch.row_seq), _ptr(batch.seq_slot), _ptr(batch.seq_q_start), _ptr(batch.seq_q_len), _stream()),
+           2 if taps > 1 else 1)
+
+
+def soft_cap_(logits: torch.Tensor, cap: float) -> None:
+    """In place: logits = cap * tanh(logits / cap), float32."""
+    _need(logits, "logits", torch.float32)
+    _check(_lib.gb_soft_cap(_ptr(logits), c_int64(logits.numel()), c_float(cap), _stream()))

@@ -1,12 +1,13 @@
 """The parts a decoder is assembled from, and their registration under their kind names."""
 from .. import registry
-from .base import (FeedForward, KVRequest, KVStateRequest, Mixer, Norm, Part, PositionEncoding, Runtime, StateRequest,
+from .base import (BlockStateRequest, FeedForward, KVRequest, KVStateRequest, Mixer, Norm, Part, PositionEncoding, Runtime, StateRequest,
                    TensorDecl)
 from .attention import Attention
 from .block import PreNormBlock
 from .delta_rule import DeltaRule
 from .dense_ff import ClampedGLU, ReluSquared
 from .diff_attention import DiffAttention
+from .forget_state import ForgetState
 from .latent_attention import LatentAttention
 from .postnorm import PostNormBlock
 from .gated_attention import GatedAttention
@@ -16,6 +17,7 @@ from .moe import MoE
 from .norm import RMSNorm
 from .reinject import Reinject
 from .rope import NoPosition, PairRotaryEmbedding, RotaryEmbedding
+from .sandwich import SandwichBlock
 from .sigmoid_attention import SigmoidAttention
 from .swiglu import SwiGLU
 
@@ -31,6 +33,7 @@ registry.register_mixer("sigmoid_attention", SigmoidAttention)
 registry.register_mixer("delta_rule", DeltaRule)
 registry.register_mixer("diff_attention", DiffAttention)
 registry.register_mixer("latent_attention", LatentAttention)
+registry.register_mixer("hgrn2", ForgetState)
 registry.register_feed_forward("swiglu", SwiGLU)
 registry.register_feed_forward("relu2_ff", ReluSquared)
 registry.register_feed_forward("glu_clamp", ClampedGLU)
@@ -38,7 +41,8 @@ registry.register_feed_forward("moe", MoE)
 registry.register_block("prenorm", PreNormBlock)
 registry.register_block("hyper", HyperBlock)
 registry.register_block("postnorm", PostNormBlock)
+registry.register_block("sandwich", SandwichBlock)
 registry.register_junction("reinject", Reinject)
 
-__all__ = ["ClampedGLU", "DiffAttention", "LatentAttention", "PostNormBlock", "ReluSquared", "Attention", "DecayState", "DeltaRule", "FeedForward", "GatedAttention", "HyperBlock", "KVStateRequest", "MatrixMemory", "MoE", "SigmoidAttention", "PairRotaryEmbedding", "KVRequest", "Mixer", "NoPosition", "Norm", "Part", "PositionEncoding",
+__all__ = ["BlockStateRequest", "ForgetState", "SandwichBlock", "ClampedGLU", "DiffAttention", "LatentAttention", "PostNormBlock", "ReluSquared", "Attention", "DecayState", "DeltaRule", "FeedForward", "GatedAttention", "HyperBlock", "KVStateRequest", "MatrixMemory", "MoE", "SigmoidAttention", "PairRotaryEmbedding", "KVRequest", "Mixer", "NoPosition", "Norm", "Part", "PositionEncoding",
            "PreNormBlock", "Reinject", "RMSNorm", "RotaryEmbedding", "Runtime", "StateRequest", "SwiGLU", "TensorDecl"]

@@ -68,6 +68,15 @@ class KVStateRequest:
     state: StateRequest
 
 
+@dataclass(frozen=True)
+class BlockStateRequest:
+    """What a block arrangement keeps for itself beside what its mixer asked for: ``mixer`` is the mixer's own
+    request (any of the above, or None) and ``state`` a further state of fixed size per sequence.  The run's view has
+    the mixer's view as ``view.mixer`` and the state as ``view.state``."""
+    mixer: object
+    state: StateRequest
+
+
 @dataclass
 class RowStats:
     """What travels between parts instead of a pending addend when the residual is already complete

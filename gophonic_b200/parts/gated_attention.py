@@ -4,7 +4,8 @@ and, optionally, another layer's keys and values (``GatedAttentionSpec``); each 
 
 Per row: q | k | v | g = x [Wq; Wk; Wv; Wg]^T in one product (a layer that reads another layer's
 cache has only q and g); biases, the norm of q and k, their position encoding and the cache write in
-one row-wise kernel; scores (q . k) * scale in float32 over the keys j <= i with i - j < window or
+one row-wise kernel (a layer whose values are its keys as projected has no v: the kernel stores the key twice, before and
+behind norm and rotation); scores (q . k) * scale in float32 over the keys j <= i with i - j < window or
 j < keep_first, softmax with one more term in the denominator; the heads, each ``value_dim`` wide,
 times sigmoid(g); out = ctx Wo^T (+ bo).  Keys are cached after rotation, so a layer that shares them
 rotates only its queries.
@@ -18,6 +19,7 @@ import torch
 from .. import registry
 from .attention import Attention
 from .base import KVRequest, Runtime, TensorDecl
+from .rope import scaled_magnitude
 
 
 class GatedAttention(Attention):
@@ -26,6 +28,11 @@ class GatedAttention(Attention):
     @staticmethod
     def _names(spec):
         return dict(spec.names)
+
+    @staticmethod
+    def _shares_key(spec) -> bool:
+        """Whether the values are the keys as projected."""
+        return bool(getattr(spec, "value_from_key", False))
 
     @classmethod
     def declare(cls, spec, prefix: str) -> List[TensorDecl]:
@@ -36,13 +43,15 @@ class GatedAttention(Attention):
         if spec.bias:
             decls.append(TensorDecl(prefix + n["q"] + spec.bias_suffix, (qd,), role="vector"))
         if spec.own_kv:
-            decls += [TensorDecl(prefix + n["k"], (kd, spec.hidden)), TensorDecl(prefix + n["v"], (vd, spec.hidden))]
-            if spec.bias:
-                decls += [TensorDecl(prefix + n["k"] + spec.bias_suffix, (kd,), role="vector"),
-                          TensorDecl(prefix + n["v"] + spec.bias_suffix, (vd,), role="vector")]
+            for key, size in (("k", kd), ("v", vd)):
+                if key == "v" and cls._shares_key(spec):
+                    continue
+                decls.append(TensorDecl(prefix + n[key], (size, spec.hidden)))
+                if spec.bias:
+                    decls.append(TensorDecl(prefix + n[key] + spec.bias_suffix, (size,), role="vector"))
         if spec.gate:
             decls.append(TensorDecl(prefix + n["g"], (od, spec.hidden)))
-        if getattr(spec, "qk_norm", None) is not None:
+        if getattr(spec, "qk_norm", None) is not None and getattr(spec, "qk_norm_weight", True):
             span = bool(getattr(spec, "qk_norm_span", False))
             decls.append(TensorDecl(prefix + n["q_norm"], (qd if span else spec.head_dim,), role="norm"))
             if spec.own_kv:
@@ -66,8 +75,14 @@ class GatedAttention(Attention):
         self.rt = runtime
         n = self._names(spec)
         parts = [tensors[prefix + n["q"]]]
+        self.value_from_key = self._shares_key(spec)
+        if self.value_from_key and (spec.bias or not spec.own_kv or spec.value_dim != spec.head_dim or getattr(spec, "qk_norm_span", False)):
+            raise ValueError(f"{prefix}: values that are the keys need keys of this layer's own, as wide as the values, without biases "
+                             f"and without a norm over the whole projection")
         if spec.own_kv:
-            parts += [tensors[prefix + n["k"]], tensors[prefix + n["v"]]]
+            parts.append(tensors[prefix + n["k"]])
+            if not self.value_from_key:
+                parts.append(tensors[prefix + n["v"]])
         if spec.gate:
             parts.append(tensors[prefix + n["g"]])
         if len({t.dtype for t in parts}) != 1:
@@ -83,7 +98,14 @@ class GatedAttention(Attention):
         self.q_norm = self.k_norm = self.sinks = self.o_bias = None
         self.eps = 0.0
         self.norm_span = bool(getattr(spec, "qk_norm_span", False))
-        if getattr(spec, "qk_norm", None) is not None:
+        if getattr(spec, "qk_norm", None) is not None and not getattr(spec, "qk_norm_weight", True):
+            # no weight: ones (a product with one changes no bit)
+            size = lambda heads: (heads if self.norm_span else 1) * spec.head_dim
+            self.q_norm = torch.ones(size(spec.heads), dtype=torch.float32, device=self.o.device)
+            if spec.own_kv:
+                self.k_norm = torch.ones(size(spec.kv_heads), dtype=torch.float32, device=self.o.device)
+            self.eps = float(spec.qk_norm.eps)
+        elif getattr(spec, "qk_norm", None) is not None:
             self.q_norm = tensors[prefix + n["q_norm"]].to(torch.float32).contiguous()
             if spec.own_kv:
                 self.k_norm = tensors[prefix + n["k_norm"]].to(torch.float32).contiguous()
@@ -93,10 +115,14 @@ class GatedAttention(Attention):
         if getattr(spec, "out_bias", False):
             self.o_bias = tensors[prefix + n["o"] + spec.bias_suffix].to(torch.float32).contiguous()
         self.position = registry.part_class("position", spec.position.kind)(spec.position, prefix, tensors, runtime)
+        if getattr(spec, "qk_norm_after", False) and (getattr(spec, "qk_norm_weight", True)
+                                                      or scaled_magnitude(getattr(spec.position, "scaling", None)) != 1.0):
+            raise ValueError(f"{prefix}: a norm behind the position encoding is built for norms without a weight and encodings that keep "
+                             f"a head's length")
         self.q_dim = spec.heads * spec.head_dim
         self.kv_heads_own = spec.kv_heads if spec.own_kv else 0
         self.k_dim = self.kv_heads_own * spec.head_dim
-        self.v_dim = self.kv_heads_own * spec.value_dim
+        self.v_dim = 0 if self.value_from_key else self.kv_heads_own * spec.value_dim
         self.o_dim = spec.heads * spec.value_dim
         self.g_off = self.q_dim + self.k_dim + self.v_dim
 
@@ -148,7 +174,8 @@ class GatedAttention(Attention):
         ops.qk_norm_rope_kv_write(qkvg, s.heads, self.kv_heads_own, s.head_dim, self.q_norm, self.k_norm, self.eps, cos, sin, rot,
                                   batch.row_pos, batch.row_seq, batch.seq_slot, cache.block_table, cache.k if s.own_kv else None,
                                   cache.v if s.own_kv else None, s.own_kv, biases=self.biases,
-                                  pairs=bool(getattr(self.position, "pairs", False)), value_dim=s.value_dim, span=self.norm_span)
+                                  pairs=bool(getattr(self.position, "pairs", False)), value_dim=s.value_dim, span=self.norm_span,
+                                  value_from_key=self.value_from_key)
         ctx = torch.empty((rows, self.o_dim), dtype=x.dtype, device=x.device)
         splits, scratch = self.key_splits(batch)
         ops.attention(qkvg, ctx, cache.k, cache.v, cache.block_table, batch.seq_slot, batch.seq_q_start, batch.seq_q_len,

@@ -8,7 +8,7 @@ kv_rank + rot_dim channels that all query heads read and whose first kv_rank cha
 cache keeps no value plane: ``KVRequest.values_in_keys``).  Nothing is expanded per cached token, so prompts in
 portions, single tokens and batches are one path.
 
-Per step: one product for both down-projections; a row-wise kernel for the two RMS norms, the rotation of k_r and the
+Per step: one product for both down-projections (and the output gate's pre-activations, if there is one); a row-wise kernel for the two RMS norms, the rotation of k_r and the
 cache write (``ops.latent_prep``); the query up-projection; the per-head product with W_uk and the rotation of the
 queries' rotated part into the absorbed queries; attention; the per-head product with W_uv; the output projection.
 The per-head products are one launch for all heads: on the CUDA cores for few rows and for float32, on the tensor cores
@@ -36,7 +36,9 @@ class LatentAttention(Mixer):
         return [TensorDecl(prefix + n["dq"], (Q, spec.hidden)), TensorDecl(prefix + n["dq_norm"], (Q,), role="norm"),
                 TensorDecl(prefix + n["uq"], (H * (d + dr), Q)), TensorDecl(prefix + n["dkv"], (R + dr, spec.hidden)),
                 TensorDecl(prefix + n["dkv_norm"], (R,), role="norm"), TensorDecl(prefix + n["uk"], (H * d, R)),
-                TensorDecl(prefix + n["uv"], (H * dv, R)), TensorDecl(prefix + n["o"], (spec.hidden, H * dv))]
+                TensorDecl(prefix + n["uv"], (H * dv, R))] + (
+                    [TensorDecl(prefix + n["g"], (H * dv, spec.hidden))] if getattr(spec, "gate", False) else []) + [
+                TensorDecl(prefix + n["o"], (spec.hidden, H * dv))]
 
     @classmethod
     def cache_request(cls, spec):
@@ -49,7 +51,13 @@ class LatentAttention(Mixer):
         dq, dkv = tensors[prefix + n["dq"]], tensors[prefix + n["dkv"]]
         if dq.dtype != dkv.dtype:
             raise ValueError(f"{prefix}: the down-projections are stored as {dq.dtype} and {dkv.dtype}; they must agree")
-        self.down = torch.cat([dq, dkv], dim=0).contiguous()          # x is read once
+        parts = [dq, dkv]
+        self.gated = bool(getattr(spec, "gate", False))
+        if self.gated:
+            parts.append(tensors[prefix + n["g"]])
+            if parts[2].dtype != dq.dtype:
+                raise ValueError(f"{prefix}: the down-projections are {dq.dtype} and the gate's matrix {parts[2].dtype}; they must agree")
+        self.down = torch.cat(parts, dim=0).contiguous()              # x is read once
         self.uq = tensors[prefix + n["uq"]].contiguous()
         uk, uv = tensors[prefix + n["uk"]], tensors[prefix + n["uv"]]
         # a head's W_uk is [head_dim, kv_rank]: as stored it maps plain query channels (K) to latent channels (N)
@@ -114,8 +122,9 @@ class LatentAttention(Mixer):
             raise ValueError("attention needs a key/value cache plane")
         if cache.k.dtype != x.dtype:
             raise ValueError(f"attention: cache holds {cache.k.dtype}, activations are {x.dtype}")
-        lat = torch.empty((rows, Q + R + dr), dtype=x.dtype, device=x.device)
-        ops.gemm(x, self.down, lat)
+        made = torch.empty((rows, self.down.shape[0]), dtype=x.dtype, device=x.device)   # [query latent | kv latent | k_r | gate]
+        ops.gemm(x, self.down, made)
+        lat = made[:, :Q + R + dr]
         cos, sin, _ = self.position.kernel_args()
         cq = torch.empty((rows, Q), dtype=x.dtype, device=x.device)
         ops.latent_prep(lat, cq, self.q_norm, self.kv_norm, float(s.eps), cos, sin, Q, R, dr, batch.row_pos, batch.row_seq, batch.seq_slot,
@@ -132,4 +141,6 @@ class LatentAttention(Mixer):
                       chunk=int(s.chunk))
         ctx = torch.empty((rows, H * dv), dtype=x.dtype, device=x.device)
         self._per_head(mixed.view(rows, H, R), self.uv_kn, self.uv_nk, ctx.view(rows, H, dv))
+        if self.gated:
+            ops.head_norm_gate(ctx, made[:, Q + R + dr:], ctx, H, dv, ops.GATE_SIGMOID)
         ops.gemm(ctx, self.o, out)

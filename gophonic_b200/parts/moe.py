@@ -4,7 +4,8 @@ weights that are not renormalised, weights that multiply an expert's input (out 
 experts down_e(silu(gate_e x) * (up_e x)), whose gate and up matrices are then stacked expert by expert as
 [gate_e; up_e] (or, ``act`` "glu_clamp", the clamped gate g sigmoid(slope g) (u + 1)), a bias on the router's logits,
 and a shared expert that every token uses (a feed-forward part of its own, whatever kind its spec names, added to the
-sum as it is or times sigmoid(w . x), one number a token; w then rides as one more row of the router's matrix).
+sum as it is or times sigmoid(w . x), one number a token; w then rides as one more row of the router's matrix), a choice
+by corrected scores (the weights come from the scores without the correction) and a choice inside the best groups of experts.
 An expert has no biases, so a weight on its input is a factor on the outputs of its first products: it is applied
 to them in float32, inside the activation between the two products.
 
@@ -42,6 +43,8 @@ class MoE(FeedForward):
         decls = [TensorDecl(prefix + "router", (spec.experts, spec.hidden))]
         if getattr(spec, "router_bias", False):
             decls.append(TensorDecl(prefix + "router" + spec.router_bias_suffix, (spec.experts,), role="vector"))
+        if getattr(spec, "correction", False):
+            decls.append(TensorDecl(prefix + spec.correction_name, (spec.experts,), role="vector"))
         for e in range(spec.experts):
             if getattr(spec, "act", "relu2") != "relu2":
                 decls.append(TensorDecl(prefix + f"e{e}.gate", (spec.intermediate, spec.hidden)))
@@ -76,6 +79,10 @@ class MoE(FeedForward):
         self.router_bias = None
         if getattr(spec, "router_bias", False):
             self.router_bias = tensors[prefix + "router" + spec.router_bias_suffix].to(torch.float32).contiguous()
+        self.correction = None
+        if getattr(spec, "correction", False):
+            self.correction = tensors[prefix + spec.correction_name].to(torch.float32).contiguous()
+        self.groups, self.keep_groups = int(getattr(spec, "groups", 1)), int(getattr(spec, "keep_groups", 1))
         shared = getattr(spec, "shared", None)
         self.shared = None if shared is None else registry.part_class("feed_forward", shared.kind)(shared, prefix + spec.shared_prefix, tensors, runtime)
         self.shared_gated = shared is not None and bool(getattr(spec, "shared_gate", False))
@@ -119,7 +126,8 @@ class MoE(FeedForward):
         dense = torch.empty((rows, s.experts), dtype=torch.float32, device=x.device)
         index = torch.empty((rows, s.top), dtype=torch.int32, device=x.device)
         weight = torch.empty((rows, s.top), dtype=torch.float32, device=x.device)
-        ops.moe_route(logits, s.top, float(s.renorm_eps), dense, index, weight, score=self.score, renorm=self.renorm)
+        ops.moe_route(logits, s.top, float(s.renorm_eps), dense, index, weight, score=self.score, renorm=self.renorm,
+                      correction=self.correction, groups=self.groups, keep_groups=self.keep_groups)
         if rows <= self.ROWS_SPARSE and s.top < s.experts:
             if rows * s.top <= s.experts:      # hardly two pairs with one expert: a pair reads its expert's matrices
                 ops.moe_rows(x, self.up, self.down, index, weight, out, s.experts, s.intermediate, weight_input=self.weight_input, **kw)

@@ -126,11 +126,13 @@ def _register_builtin() -> None:
     from .config.vepitar import VepitarConfig
     from .config.kalonex import KalonexConfig
     from .config.kimilix import KimilixConfig
+    from .config.zenorax import ZenoraxConfig
     register_architecture("Qwen3ForCausalLM", Qwen3Config, model_type="qwen3")
     register_architecture("Pugalix", PugalixConfig)
     register_architecture("Vepitar", VepitarConfig)
     register_architecture("Kalonex", KalonexConfig)
     register_architecture("Kimilix", KimilixConfig)
+    register_architecture("Zenorax", ZenoraxConfig)
 
 
 _register_builtin()
