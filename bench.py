@@ -617,6 +617,107 @@ def probe(name, **opts):
             work, unit = 2.0 * heads * (d + dv) * seen, "TFLOP/s"
         else:
             work, unit = float(nseq) * (seen_keys + 64) * key_bytes, "GB/s"
+    elif name in ("forget_scan_prompt", "forget_step_b64"):
+        # the recurrence whose forget gate writes, sizes as for state_scan_prompt / state_step_b64 (a repeated prompt call takes
+        # its own activations as pre-activations: other numbers, the same cost)
+        heads, d = 16, 128
+        prompt = name.endswith("prompt")
+        nseq, q_len = (1, 2048) if prompt else (64, 1)
+        rows = nseq * q_len
+        f32 = lambda *shape: torch.randn(*shape, device=dev, generator=g)
+        rows_qvf = f32(rows, 3 * heads * d)
+        bias, low = f32(heads * d), torch.rand(heads * d, device=dev, generator=g)
+        state = torch.zeros((nseq, heads, d * d), dtype=torch.float32, device=dev)
+        out = torch.empty((rows, heads * d), dtype=torch.float32, device=dev)
+        ints = lambda x: torch.tensor(x, dtype=torch.int32, device=dev)
+        slot, start, ql = ints(list(range(nseq))), ints([i * q_len for i in range(nseq)]), ints([q_len] * nseq)
+
+        def fn():
+            ops.state_scan(rows_qvf, 0, 0, heads * d, heads, d, d, 1.0, state, out, slot, start, ql, nseq, decay=rows_qvf[:, 2 * heads * d:],
+                           gate_bias=bias, lower=low, max_q_len=q_len)
+        if prompt:
+            work, unit = float(rows) * heads * d * d, "state updates/s"
+        else:
+            work, unit = 2.0 * state.numel() * 4, "GB/s"
+    elif name in ("sandwich_mid", "sandwich_open_4", "sandwich_open_8", "norm_scale_add_rows", "conv_rows_prompt", "conv_qkv_prompt"):
+        # row-wise kernels over 16384 rows of 2048 (each operand is as large as L2): a sublayer's output joined and normed; the
+        # same with a weighted sum over 4 or 8 planes; the postnorm block's kernel; the convolutions ahead of a mixer
+        from types import SimpleNamespace
+        rows, W, taps = 16384, 2048, 4
+        f32 = lambda *shape: torch.randn(*shape, device=dev, generator=g)
+        ints = lambda x: torch.tensor(x, dtype=torch.int32, device=dev)
+        y, base, w = f32(rows, W), f32(rows, W), torch.ones(W, device=dev)
+        x = torch.empty((rows, W), dtype=bf, device=dev)
+        unit = "GB/s"
+        nseq = 8
+        packed = SimpleNamespace(nseq=nseq, max_q_len=rows // nseq, row_seq=ints([i // (rows // nseq) for i in range(rows)]),
+                                 row_pos=ints([i % (rows // nseq) for i in range(rows)]), seq_slot=ints(list(range(nseq))),
+                                 seq_q_start=ints([i * (rows // nseq) for i in range(nseq)]), seq_q_len=ints([rows // nseq] * nseq))
+        if name == "norm_scale_add_rows":
+            work = rows * W * (4 + 4 + 4 + 2)
+            fn = lambda: ops.norm_scale_add(base, y, w, 1e-6, x)
+        elif name == "sandwich_mid":
+            result = torch.empty_like(base)
+            work = rows * W * (4 + 4 + 4 + 2)
+            fn = lambda: ops.sandwich_rows(base=base, y=y, y_weight=w, y_eps=1e-6, result=result, out=x, norm_weight=w, eps=1e-6)
+        elif name.startswith("sandwich_open"):
+            n = int(name.rsplit("_", 1)[1])
+            planes, avg, x_out, normed = f32(n + 1, rows, W), torch.ones(n + 1, device=dev), torch.empty_like(base), torch.empty_like(base)
+            work = rows * W * 4 * (n + 2 + 3)
+            fn = lambda: ops.sandwich_rows(base=planes[n], y=y, y_weight=w, y_eps=1e-6, result=planes[n], planes=planes, n_planes=n, average=avg,
+                                           x_out=x_out, out=normed, norm_weight=w, eps=1e-6)
+        elif name == "conv_rows_prompt":
+            conv, state = f32(taps, W), torch.zeros((nseq, (taps - 1) * W), device=dev)
+            work = rows * W * (4 + 2)
+            fn = lambda: ops.conv_rows(base, conv, state, x, packed)
+        else:
+            heads, kvh, d = 8, 4, 128                    # as many channels: 8 + 4 + 4 heads of 128
+            qkv, q = rnd(rows, W), torch.empty((rows, heads * d), dtype=bf, device=dev)
+            pages = rows // 64
+            k, v = rnd(pages, kvh, 64, d), rnd(pages, kvh, 64, d)
+            table = torch.arange(pages, dtype=torch.int32, device=dev).reshape(nseq, pages // nseq)
+            conv, state = f32(W, taps), torch.zeros((nseq, (taps - 1) * W), device=dev)
+            work = rows * W * (2 + 2)
+            fn = lambda: ops.conv_qkv(qkv, q, heads, kvh, d, d, conv, state, True, False, 1e-6, packed, table, k, v)
+    elif name in ("moe_few_relu2", "moe_few_clamped", "moe_prompt_relu2", "moe_prompt_clamped"):
+        # a mixture of 16 experts, width 2048: 4 experts of 1536 a token without a gate, or 2 gated ones of 2048 (as many rows read a
+        # token); 8 single tokens (bound by reading the chosen experts' matrices) or a prompt of 2048
+        from gophonic_b200.config.spec import MoESpec
+        from gophonic_b200.engine.model import make_runtime
+        from gophonic_b200.parts.moe import MoE
+        W, E, rows = 2048, 16, 8 if "few" in name else 2048
+        top, ff, act = (4, 1536, "relu2") if name.endswith("relu2") else (2, 2048, "glu_clamp")
+        spec = MoESpec(hidden=W, experts=E, top=top, intermediate=ff, renorm_eps=0.0, score="sigmoid" if act == "relu2" else "softmax",
+                       renorm=act != "relu2", act=act, act_limit=7.0, act_slope=1.702, correction=act == "relu2", groups=4 if act == "relu2" else 1,
+                       keep_groups=2 if act == "relu2" else 1)
+        part = MoE(spec, "", {d.name: (torch.zeros(d.shape, device=dev).to(bf) if d.role == "vector" else rnd(*d.shape, scale=0.02)) for d in
+                              MoE.declare(spec, "")}, make_runtime("bfloat16", dev))
+        x, out = rnd(rows, W), torch.empty((rows, W), device=dev)
+
+        def fn():
+            part.forward(None, x, out)
+        per = (1 if act == "relu2" else 2) + 1
+        if rows == 8:
+            # in a graph, as a decode step runs it; four parts take turns so that the matrices come from memory
+            parts = [part] + [MoE(spec, "", {d.name: (torch.zeros(d.shape, device=dev).to(bf) if d.role == "vector" else rnd(*d.shape, scale=0.02)) for d in
+                                             MoE.declare(spec, "")}, make_runtime("bfloat16", dev)) for _ in range(3)]
+            logits = torch.empty((rows, E), device=dev)
+            ops.gemm(x, part.router, logits)
+            index = torch.empty((rows, top), dtype=torch.int32, device=dev)
+            ops.moe_route(logits, top, 0.0, torch.empty((rows, E), device=dev), index, torch.empty((rows, top), device=dev), score=spec.score,
+                          renorm=spec.renorm, groups=spec.groups, keep_groups=spec.keep_groups)
+            used = len(set(index.flatten().tolist()))
+            for q in parts:
+                q.forward(None, x, out)
+            torch.cuda.synchronize()
+            graph = torch.cuda.CUDAGraph()
+            with torch.cuda.graph(graph):
+                for q in parts:
+                    q.forward(None, x, out)
+            fn = graph.replay
+            work, unit = 4.0 * used * per * ff * W * 2, "GB/s"
+        else:
+            work, unit = 2.0 * rows * top * per * ff * W, "TFLOP/s"
     elif name in ("prefill_step", "decode_step"):
         # a whole engine step of a 4-layer model with the layer sizes of the benchmark (or of --model):
         # the launch list of a profiler then shows every kernel of a layer with its share.  --batch

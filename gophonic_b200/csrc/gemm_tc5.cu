@@ -685,6 +685,8 @@ __global__ void __launch_bounds__(THREADS) gemm_tc5_grouped_kernel(const __grid_
 
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int KT = (K + BK - 1) / BK;
+    const bool square = gated == 3;      // no gate: every output is squared where it is positive
+    if (square) gated = 0;
     const int TN = gated ? BN / 2 : BN;  // outputs a tile makes
     const int tiles_n = (N + TN - 1) / TN;
 
@@ -812,6 +814,13 @@ __global__ void __launch_bounds__(THREADS) gemm_tc5_grouped_kernel(const __grid_
                     tmem_ld32(t_addr + (uint32_t)(BN / 2 + c0), u);
                     if (mine) store_gated32<TC>(C + (int64_t)crow * ldc + n0 + c0, N - (n0 + c0), vec_ok, r, u, f, gated, act_limit, act_slope);
                 } else {
+                    if (square) {
+#pragma unroll
+                        for (int e = 0; e < 32; e++) {
+                            const float v = fmaxf(__uint_as_float(r[e]), 0.f);
+                            r[e] = __float_as_uint(v * v);
+                        }
+                    }
                     store_cols32<TC>(C, ldc, crow, mine ? 0x7fffffff : 0, N, n0 + c0, r, 0, vec_ok);
                 }
             }
@@ -853,7 +862,7 @@ int launch_grouped(const void* A, const void* W, void* C, const int* offsets, in
         if (cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev) != cudaSuccess || sms <= 0) sms = 148;
     }
     // the groups' sizes are not known here: every group may end with a tile that is partly empty
-    const int tn = gated ? BN / 2 : BN;
+    const int tn = gated == 1 || gated == 2 ? BN / 2 : BN;
     const int64_t most = ((int64_t)ceil_div(P, BM) + (groups < P ? groups : P)) * ceil_div(N, tn);
     const int grid = most < sms ? (int)most : sms;
     cudaError_t e = launch_pdl(gemm_tc5_grouped_kernel<TC>, dim3(grid), dim3(THREADS), (size_t)smem, stream, map_a, map_w, (TC*)C, offsets,
@@ -941,17 +950,17 @@ GB_API int gb_gemm_tc5_grouped(const void* A, const void* W, void* C, int c_dtyp
 }
 
 // The same with the gate's kind: gated 1: silu(f g) * (f u); gated 2: c sigmoid(slope c) (v + 1) with c = min(f g, limit) and
-// v = clamp(f u, -limit, limit).
+// v = clamp(f u, -limit, limit).  gated 3: blocks of N rows, no gate, C = max(sum, 0)^2.
 GB_API int gb_gemm_tc5_grouped_act(const void* A, const void* W, void* C, int c_dtype, const int* offsets, int groups, int P, int N, int K,
                                    int64_t lda, int64_t ldw, int64_t ldc, int w_rows, int by_cols, int gated, const float* row_weight,
                                    const int* row_map, float act_limit, float act_slope, cudaStream_t stream) {
-    if (gated < 0 || gated > 2) GB_REFUSE("gemm_tc5_grouped: unknown gate %d", gated);
+    if (gated < 0 || gated > 3) GB_REFUSE("gemm_tc5_grouped: unknown gate %d", gated);
     if (P <= 0 || N <= 0 || groups <= 0) return 0;
     if (K <= 0 || (K & 7)) GB_REFUSE("gemm_tc5_grouped: K = %d must be a positive multiple of 8", K);
     if ((lda & 7) || lda < K) GB_REFUSE("gemm_tc5_grouped: row stride %lld of A must be a multiple of 8 and at least K", (long long)lda);
     if ((ldw & 7) || ldw < (by_cols ? (int64_t)groups * K : (int64_t)K))
         GB_REFUSE("gemm_tc5_grouped: row stride %lld of W must be a multiple of 8 and hold its blocks", (long long)ldw);
-    if (!by_cols && w_rows < (gated ? 2 * N : N)) GB_REFUSE("gemm_tc5_grouped: a block of %d rows does not hold %d outputs", w_rows, N);
+    if (!by_cols && w_rows < (gated == 1 || gated == 2 ? 2 * N : N)) GB_REFUSE("gemm_tc5_grouped: a block of %d rows does not hold %d outputs", w_rows, N);
     if (by_cols && gated) GB_REFUSE("gemm_tc5_grouped: gated outputs come from blocks of rows");
     if ((int64_t)groups * (by_cols ? K : w_rows) > 0x7fffffff) GB_REFUSE("gemm_tc5_grouped: W is too large");
     if (ldc < N) GB_REFUSE("gemm_tc5_grouped: row stride %lld of C is shorter than N = %d", (long long)ldc, N);

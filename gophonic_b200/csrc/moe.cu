@@ -17,6 +17,9 @@
 // moe_up_rows / moe_down_rows: the same feed-forward for a step of few rows, reading only the chosen
 // experts' matrices (a warp a hidden unit, or an output column, of one (row, choice) pair).
 //
+// moe_up_grouped / moe_down_grouped: the same with the pairs sorted by expert, so an expert's matrices are read once; on the
+// tensor cores where rows are aligned.
+//
 // moe_group / moe_gather / relu2 / moe_combine: a step of many rows sorts its (row, choice) pairs by expert
 // (counts, offsets, and each pair's place in the sorted order), gathers the rows in that order so that every
 // expert's rows lie together for one product an expert, squares the positive part between the two products, and
@@ -24,6 +27,7 @@
 // expert's group may differ from run to run; a row's result does not depend on it.
 #include "api.h"
 #include "common.cuh"
+#include "mma.cuh"
 
 #include <math.h>
 
@@ -296,6 +300,125 @@ __global__ void __launch_bounds__(128) moe_down_grouped_kernel(MoeRowsParams p, 
     }
 }
 
+// The same two products in bfloat16 on the tensor cores: a CTA takes 16 rows of ONE expert's matrix (16 hidden units, or 16
+// output columns), streams them once from global memory straight into mma.sync fragments (the fragment's k order is the
+// memory's: see gemm_skinny.cu) and multiplies them with eight of the expert's pairs at a time; its warps split K and
+// meet in shared memory, added in warp order, so a pair's sums do not depend on what else the step holds.
+constexpr int MG_WARPS = 8;
+
+// W: this lane's two rows (g and g + 8 of the tile) at its place in a 32-wide step, X: its pair's row at the same place
+__device__ __forceinline__ void stream_product(float (&acc)[4], const __nv_bfloat16* __restrict__ w_lo, const __nv_bfloat16* __restrict__ w_hi,
+                                               const __nv_bfloat16* __restrict__ x, int k, int k_end, int t) {
+    const int k_full = k + (k_end - k) / 32 * 32;
+    constexpr int U = 4;
+    for (; k + U * 32 <= k_full; k += U * 32) {      // the loads of four steps are in flight before the first product needs one
+        uint4 a_lo[U], a_hi[U], b[U];
+#pragma unroll
+        for (int u = 0; u < U; u++) {
+            a_lo[u] = ld_stream16(w_lo + k + u * 32);
+            a_hi[u] = ld_stream16(w_hi + k + u * 32);
+        }
+#pragma unroll
+        for (int u = 0; u < U; u++) b[u] = *reinterpret_cast<const uint4*>(x + k + u * 32);
+#pragma unroll
+        for (int u = 0; u < U; u++) {
+            mma_bf16_16816(acc, a_lo[u].x, a_hi[u].x, a_lo[u].y, a_hi[u].y, b[u].x, b[u].y);
+            mma_bf16_16816(acc, a_lo[u].z, a_hi[u].z, a_lo[u].w, a_hi[u].w, b[u].z, b[u].w);
+        }
+    }
+    for (; k < k_full; k += 32) {
+        const uint4 a_lo = ld_stream16(w_lo + k), a_hi = ld_stream16(w_hi + k), b = *reinterpret_cast<const uint4*>(x + k);
+        mma_bf16_16816(acc, a_lo.x, a_hi.x, a_lo.y, a_hi.y, b.x, b.y);
+        mma_bf16_16816(acc, a_lo.z, a_hi.z, a_lo.w, a_hi.w, b.z, b.w);
+    }
+    if (k < k_end) {      // K is a multiple of 8: a lane's piece is wholly inside or wholly outside
+        const bool in = k + t * 8 < k_end;
+        const uint4 z = make_uint4(0, 0, 0, 0);
+        const uint4 a_lo = in ? ld_stream16(w_lo + k) : z, a_hi = in ? ld_stream16(w_hi + k) : z, b = in ? *reinterpret_cast<const uint4*>(x + k) : z;
+        mma_bf16_16816(acc, a_lo.x, a_hi.x, a_lo.y, a_hi.y, b.x, b.y);
+        mma_bf16_16816(acc, a_lo.z, a_hi.z, a_lo.w, a_hi.w, b.z, b.w);
+    }
+}
+
+__device__ __forceinline__ void leave_fragment(float* __restrict__ mine, const float (&acc)[4], int g, int t) {
+    mine[g * 8 + 2 * t] = acc[0];
+    mine[g * 8 + 2 * t + 1] = acc[1];
+    mine[(g + 8) * 8 + 2 * t] = acc[2];
+    mine[(g + 8) * 8 + 2 * t + 1] = acc[3];
+}
+
+template <bool GATED>
+__global__ void __launch_bounds__(32 * MG_WARPS) moe_up_grouped_mma_kernel(MoeRowsParams p, const int* __restrict__ offsets,
+                                                                           const int* __restrict__ src_row) {
+    __shared__ float red[GATED ? 2 : 1][MG_WARPS][16 * 8];
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
+    const int n0 = blockIdx.x * 16, e = blockIdx.y, K = p.hidden;
+    const int lo = offsets[e], hi = offsets[e + 1];
+    if (lo == hi) return;
+    const int i_lo = min(n0 + g, p.ff - 1), i_hi = min(n0 + g + 8, p.ff - 1);      // rows past the end repeat the last one and are dropped
+    const __nv_bfloat16* w = (const __nv_bfloat16*)p.up + (int64_t)e * (GATED ? 2 : 1) * p.ff * K + t * 8;
+    const __nv_bfloat16 *w_lo = w + (int64_t)i_lo * K, *w_hi = w + (int64_t)i_hi * K;
+    const int per = ((K + 31) / 32 + MG_WARPS - 1) / MG_WARPS * 32;
+    const int k0 = warp * per, k1 = min(k0 + per, K);
+    for (int p0 = lo; p0 < hi; p0 += 8) {
+        const __nv_bfloat16* x = (const __nv_bfloat16*)p.x + (int64_t)src_row[min(p0 + g, hi - 1)] * p.x_stride + t * 8;
+        float acc[4] = {0.f, 0.f, 0.f, 0.f}, acc2[4] = {0.f, 0.f, 0.f, 0.f};
+        if (k0 < k1) stream_product(acc, w_lo, w_hi, x, k0, k1, t);
+        if (GATED && k0 < k1) stream_product(acc2, w_lo + (int64_t)p.ff * K, w_hi + (int64_t)p.ff * K, x, k0, k1, t);
+        leave_fragment(red[0][warp], acc, g, t);
+        if (GATED) leave_fragment(red[GATED ? 1 : 0][warp], acc2, g, t);
+        __syncthreads();
+        if (threadIdx.x < 128) {
+            const int b = threadIdx.x >> 4, i = threadIdx.x & 15, at = p0 + b;
+            if (at < hi && n0 + i < p.ff) {
+                float s = 0.f, u = 0.f;
+#pragma unroll
+                for (int ww = 0; ww < MG_WARPS; ww++) {
+                    s += red[0][ww][i * 8 + b];
+                    if (GATED) u += red[GATED ? 1 : 0][ww][i * 8 + b];
+                }
+                // the same roundings as the kernel above
+                s = __bfloat162float(__float2bfloat16_rn(s));
+                u = __bfloat162float(__float2bfloat16_rn(u));
+                ((__nv_bfloat16*)p.act)[(int64_t)at * p.ff + n0 + i] =
+                    __float2bfloat16_rn(expert_act(s, u, p.weight_input ? p.weight[at] : 1.f, p.act_kind, p.weight_input, p.limit, p.slope));
+            }
+        }
+        __syncthreads();
+    }
+}
+
+__global__ void __launch_bounds__(32 * MG_WARPS) moe_down_grouped_mma_kernel(MoeRowsParams p, const int* __restrict__ offsets, float* __restrict__ ys) {
+    __shared__ float red[MG_WARPS][16 * 8];
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
+    const int n0 = blockIdx.x * 16, e = blockIdx.y, K = p.ff;
+    const int lo = offsets[e], hi = offsets[e + 1];
+    if (lo == hi) return;
+    const int64_t ldw = (int64_t)p.experts * K;
+    const int c_lo = min(n0 + g, p.hidden - 1), c_hi = min(n0 + g + 8, p.hidden - 1);
+    const __nv_bfloat16* w = (const __nv_bfloat16*)p.down + (int64_t)e * K + t * 8;
+    const __nv_bfloat16 *w_lo = w + c_lo * ldw, *w_hi = w + c_hi * ldw;
+    const int per = ((K + 31) / 32 + MG_WARPS - 1) / MG_WARPS * 32;
+    const int k0 = warp * per, k1 = min(k0 + per, K);
+    for (int p0 = lo; p0 < hi; p0 += 8) {
+        const __nv_bfloat16* x = (const __nv_bfloat16*)p.act + (int64_t)min(p0 + g, hi - 1) * K + t * 8;
+        float acc[4] = {0.f, 0.f, 0.f, 0.f};
+        if (k0 < k1) stream_product(acc, w_lo, w_hi, x, k0, k1, t);
+        leave_fragment(red[warp], acc, g, t);
+        __syncthreads();
+        if (threadIdx.x < 128) {
+            const int b = threadIdx.x >> 4, i = threadIdx.x & 15, at = p0 + b;
+            if (at < hi && n0 + i < p.hidden) {
+                float s = 0.f;
+#pragma unroll
+                for (int ww = 0; ww < MG_WARPS; ww++) s += red[ww][i * 8 + b];
+                ys[(int64_t)at * p.hidden + n0 + i] = s;
+            }
+        }
+        __syncthreads();
+    }
+}
+
 constexpr int GROUP_THREADS = 1024;
 constexpr int GROUP_MAX_EXPERTS = 512;
 
@@ -487,7 +610,16 @@ GB_API int gb_moe_rows_grouped(const MoeRowsParams* pp, const int* offsets, cons
     if (p.experts <= 0 || p.experts > 65535 || p.top <= 0 || p.ff <= 0 || p.hidden <= 0) GB_REFUSE("moe_rows: %d experts, %d a token, %d x %d", p.experts, p.top, p.ff, p.hidden);
     if (!p.x || !p.up || !p.down || !p.act || !offsets || !src_row || !ys || (p.weight_input && !p.weight)) GB_REFUSE("moe_rows: a tensor is missing");
     dim3 ugrid((p.ff + 3) / 4, p.experts), dgrid((p.hidden + 3) / 4, p.experts);
-    if (dtype == GB_BF16 && w_dtype == GB_BF16) {
+    const bool aligned = !(p.hidden & 7) && !(p.ff & 7) && !(p.x_stride & 7) &&
+                         !(((uintptr_t)p.x | (uintptr_t)p.up | (uintptr_t)p.down | (uintptr_t)p.act) & 15);
+    if (dtype == GB_BF16 && w_dtype == GB_BF16 && aligned) {
+        dim3 um((p.ff + 15) / 16, p.experts), dm((p.hidden + 15) / 16, p.experts);
+        if (p.act_kind != 0)
+            moe_up_grouped_mma_kernel<true><<<um, 32 * MG_WARPS, 0, stream>>>(p, offsets, src_row);
+        else
+            moe_up_grouped_mma_kernel<false><<<um, 32 * MG_WARPS, 0, stream>>>(p, offsets, src_row);
+        moe_down_grouped_mma_kernel<<<dm, 32 * MG_WARPS, 0, stream>>>(p, offsets, ys);
+    } else if (dtype == GB_BF16 && w_dtype == GB_BF16) {
         moe_up_grouped_kernel<__nv_bfloat16, __nv_bfloat16><<<ugrid, 128, 0, stream>>>(p, offsets, src_row);
         moe_down_grouped_kernel<__nv_bfloat16, __nv_bfloat16><<<dgrid, 128, 0, stream>>>(p, offsets, ys);
     } else if (dtype == GB_F32 && w_dtype == GB_F32) {

@@ -251,6 +251,58 @@ __global__ void __launch_bounds__(256) conv_rows_kernel(const float* __restrict_
     }
 }
 
+// The same for convolutions of few taps on rows that vectors fit: a thread owns four channels of CONV_ROWS consecutive
+// packed rows and loads them, and the TAPS - 1 rows ahead of them, once; a tap that reaches ahead of its sequence's portion
+// takes the state instead.
+constexpr int CONV_ROWS = 8;
+
+template <typename TO, int TAPS>
+__global__ void __launch_bounds__(256) conv_rows_window_kernel(const float* __restrict__ h, const float* __restrict__ conv_w,
+                                                               const float* __restrict__ state, int64_t state_slot_stride, int max_slots,
+                                                               TO* __restrict__ out, int rows, int n, const int* __restrict__ row_seq,
+                                                               const int* __restrict__ seq_slot, const int* __restrict__ seq_q_start) {
+    pdl_wait();
+    pdl_trigger();
+    const int c = (blockIdx.y * 256 + threadIdx.x) * 4;
+    const int64_t r0 = (int64_t)blockIdx.x * CONV_ROWS;
+    if (c >= n) return;
+    float x[CONV_ROWS + TAPS - 1][4], w[TAPS][4];
+    int seq[CONV_ROWS];
+#pragma unroll
+    for (int i = 0; i < CONV_ROWS + TAPS - 1; i++) {
+        const int64_t r = r0 + i - (TAPS - 1);
+        if (r >= 0 && r < rows) load_v<4>(h + r * n + c, x[i]);
+    }
+#pragma unroll
+    for (int j = 0; j < TAPS; j++) load_v<4>(conv_w + (int64_t)j * n + c, w[j]);
+#pragma unroll
+    for (int i = 0; i < CONV_ROWS; i++) seq[i] = r0 + i < rows ? row_seq[r0 + i] : 0;
+#pragma unroll
+    for (int i = 0; i < CONV_ROWS; i++) {
+        if (r0 + i >= rows) continue;
+        const int local = (int)(r0 + i - seq_q_start[seq[i]]);
+        float a[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+        for (int j = 0; j < TAPS; j++) {
+            const int back = TAPS - 1 - j;
+            float t[4];
+#pragma unroll
+            for (int u = 0; u < 4; u++) t[u] = x[i + j][u];
+            if (back > local) {
+                int slot = seq_slot[seq[i]];
+                if (!gb_check(slot, max_slots, GB_CHECK_SLOT)) slot = 0;
+                load_v<4>(state + (int64_t)slot * state_slot_stride + (int64_t)(TAPS - 1 + local - back) * n + c, t);
+            }
+#pragma unroll
+            for (int u = 0; u < 4; u++) a[u] = fmaf(w[j][u], t[u], a[u]);
+        }
+        float o[4];
+#pragma unroll
+        for (int u = 0; u < 4; u++) o[u] = x[i + TAPS - 1][u] + a[u];
+        store_v<4>(out + (r0 + i) * n + c, o);
+    }
+}
+
 // the last taps - 1 rows of every sequence's portion into its state; a portion shorter than that pushes the older rows on
 __global__ void conv_rows_state_kernel(const float* __restrict__ h, int taps, float* __restrict__ state, int64_t state_slot_stride, int max_slots,
                                        int n, const int* __restrict__ seq_slot, const int* __restrict__ seq_q_start,
@@ -299,16 +351,29 @@ GB_API int gb_conv_rows(const float* h, const float* conv_w, int taps, float* st
     if (taps > 1 && (!state || state_slot_stride < (int64_t)(taps - 1) * width)) GB_REFUSE("conv_rows: the state has no room for %d rows of %d", taps - 1, width);
     if (nseq > 65535) GB_REFUSE("conv_rows: %d sequences exceed one launch", nseq);
     const bool vec = !(width & 3) && !(((uintptr_t)h | (uintptr_t)conv_w | (uintptr_t)state | (uintptr_t)out) & 15) && !(state_slot_stride & 3);
+#define GB_WINDOW(TO, TAPS)                                                                                                                          \
+    launch_pdl(conv_rows_window_kernel<TO, TAPS>, dim3(ceil_div(rows, CONV_ROWS), ceil_div(width, 1024)), dim3(256), 0, stream, h, conv_w,            \
+               (const float*)state, state_slot_stride, max_slots, (TO*)out, rows, width, row_seq, seq_slot, seq_q_start)
+#define GB_WINDOWS(TO)                       \
+    switch (taps) {                          \
+        case 2: GB_WINDOW(TO, 2); break;     \
+        case 3: GB_WINDOW(TO, 3); break;     \
+        default: GB_WINDOW(TO, 4); break;    \
+    }
 #define GB_CONV(TO, V) \
     conv_rows_kernel<TO, V><<<rows, 256, 0, stream>>>(h, conv_w, taps, state, state_slot_stride, max_slots, (TO*)out, width, row_seq, seq_slot, seq_q_start)
-    if (out_dtype == GB_F32) {
+    const bool window = vec && taps >= 2 && taps <= 4 && rows >= 64 && ceil_div(width, 1024) <= 65535;
+    if (out_dtype != GB_F32 && out_dtype != GB_BF16) GB_REFUSE("conv_rows: unknown dtype %d", out_dtype);
+    if (window) {
+        if (out_dtype == GB_F32) GB_WINDOWS(float) else GB_WINDOWS(__nv_bfloat16)
+    } else if (out_dtype == GB_F32) {
         if (vec) GB_CONV(float, 4); else GB_CONV(float, 1);
-    } else if (out_dtype == GB_BF16) {
-        if (vec) GB_CONV(__nv_bfloat16, 4); else GB_CONV(__nv_bfloat16, 1);
     } else {
-        GB_REFUSE("conv_rows: unknown dtype %d", out_dtype);
+        if (vec) GB_CONV(__nv_bfloat16, 4); else GB_CONV(__nv_bfloat16, 1);
     }
 #undef GB_CONV
+#undef GB_WINDOWS
+#undef GB_WINDOW
     GB_CHECK_LAUNCH("conv_rows");
     if (taps > 1) {
         conv_rows_state_kernel<<<dim3(ceil_div(width, 256), nseq), 256, 0, stream>>>(h, taps, state, state_slot_stride, max_slots, width, seq_slot,

@@ -1487,7 +1487,8 @@ def gemm_grouped(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, offsets: t
     ``by_cols`` False: ``w`` is [groups * block, K] and block e its rows e * block ..; with ``gated`` a block is N gate
     rows, then N up rows, and out = silu(f g) * (f u), f = ``row_weight[row]`` (1 if absent), or with ``gate`` "glu_clamp"
     c * sigmoid(slope * c) * (v + 1), c = min(f g, limit), v = clamp(f u, -limit, limit).  ``by_cols`` True: ``w`` is
-    [N, groups * K] and block e its columns e * K ...  ``out`` is [*, N]; with ``row_map`` (int32 [P]) the result of
+    [N, groups * K] and block e its columns e * K ...  ``gate`` "relu2" (with ``gated`` False): every sum is squared where it
+    is positive and zero elsewhere.  ``out`` is [*, N]; with ``row_map`` (int32 [P]) the result of
     row r is written to row ``row_map[r]`` of ``out``, otherwise to row r."""
     _need(a, "grouped gemm a", torch.bfloat16, 2, contiguous=False)
     _need(w, "grouped gemm w", torch.bfloat16, 2, contiguous=False)
@@ -1515,11 +1516,11 @@ def gemm_grouped(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, offsets: t
         _need(row_map, "row map", torch.int32, 1)
         if row_map.numel() < P:
             raise KernelError(f"gemm_grouped: {row_map.numel()} mapped rows for {P}")
-    if gate not in ("swiglu", "glu_clamp"):
+    if gate not in ("swiglu", "glu_clamp", "relu2") or (gate == "relu2" and (gated or by_cols)):
         raise KernelError(f"gemm_grouped: unknown gate '{gate}'")
     _check(_lib.gb_gemm_tc5_grouped_act(_ptr(a), _ptr(w), _ptr(out), _code(out.dtype), _ptr(offsets), c_int(groups), c_int(P), c_int(N), c_int(K),
                                         c_int64(a.stride(0)), c_int64(w.stride(0)), c_int64(out.stride(0)), c_int(block), c_int(1 if by_cols else 0),
-                                        c_int(0 if not gated else (2 if gate == "glu_clamp" else 1)), _ptr(row_weight), _ptr(row_map),
+                                        c_int((3 if gate == "relu2" else 0) if not gated else (2 if gate == "glu_clamp" else 1)), _ptr(row_weight), _ptr(row_map),
                                         c_float(limit), c_float(slope), _stream()))
 
 

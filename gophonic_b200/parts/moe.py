@@ -173,15 +173,18 @@ class MoE(FeedForward):
             ops.gemm_grouped(xs, self.up, act, offsets, s.experts, gated=True, row_weight=sorted_w, gate=self.act, limit=self.limit, slope=self.slope)
         else:
             act = torch.empty((pairs, per), dtype=x.dtype, device=x.device)
+            squared = one_launch and not self.weight_input      # relu(z)^2 in the product's own epilogue
             if one_launch:
-                ops.gemm_grouped(xs, self.up, act, offsets, s.experts)
+                ops.gemm_grouped(xs, self.up, act, offsets, s.experts, **(dict(gate="relu2") if squared else {}))
             else:
                 bounds = offsets.tolist()       # the one host read of such a step
                 for e in range(s.experts):
                     lo, hi = bounds[e], bounds[e + 1]
                     if hi > lo:
                         ops.gemm_w_cols(xs[lo:hi], self.up[e * per:(e + 1) * per], act[lo:hi])
-            if self.act == "relu2" and not self.weight_input:
+            if squared:
+                pass
+            elif self.act == "relu2" and not self.weight_input:
                 ops.relu2(act)
             else:
                 # every sorted pair is a row of one "expert" here: its own weight (or 1), its own activation

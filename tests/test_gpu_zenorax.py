@@ -79,7 +79,7 @@ CONFIGS = {
     # tap, one head, one expert, every expert used, groups of one expert, a width that no vector load fits
     "odd": config([attention(heads=3, kv_heads=None, dim=12, rot=None, vdim=False, mlp=moe(1, 1, 56, None)),
                    latent(heads=1, dim=20, rot_dim=0, vdim=17, q_rank=7, kv_rank=9, scale=1.0, mlp=moe(5, 3, 8, 5, 4)),
-                   hgrn2(heads=1, dim=1, vdim=5, mlp=moe(3, 3, 8, 1, 1)), latent(heads=5, dim=6, rot_dim=2, vdim=10, q_rank=48, kv_rank=5, scaling=None),
+                   hgrn2(heads=1, dim=3, vdim=5, mlp=moe(3, 3, 8, 1, 1)), latent(heads=5, dim=6, rot_dim=2, vdim=10, q_rank=48, kv_rank=5, scaling=None),
                    hgrn2(heads=7, dim=20, vdim=33)], width=45, vocab=61, emb=1.0, eps=1e-6, taps=1, cap=None),
     # more taps than a short portion has tokens
     "taps": config([hgrn2(), attention()], taps=7, width=52),
@@ -448,7 +448,7 @@ def test_the_convolution_in_portions_and_token_by_token(taps, width):
     from gophonic_b200 import ops
     ops.use_device(0)
     rng = np.random.default_rng(taps)
-    lengths = [40, 23]
+    lengths = [90, 103]
     h = [rng.standard_normal((n, width)) for n in lengths]
     conv = _f32(0.4 * rng.standard_normal((taps, width)))
     hs = [_f32(a) for a in h]
@@ -456,7 +456,7 @@ def test_the_convolution_in_portions_and_token_by_token(taps, width):
     ones = torch.ones(width, dtype=torch.float32, device="cuda:0")
     state = torch.zeros((3, max(taps - 1, 1) * width), dtype=torch.float32, device="cuda:0")
     got, at, slots = [[], []], [0, 0], [2, 0]
-    for portion in ([3, 5], [2, 2], [1, 4], [20, 1], [2, 2]):
+    for portion in ([3, 5], [2, 2], [1, 4], [20, 1], [2, 2], [40, 50], [2, 30]):      # few rows a step, and many (another kernel)
         x = torch.cat([hs[s][at[s]:at[s] + n] for s, n in enumerate(portion)]).contiguous()
         out = torch.zeros_like(x)
         ops.conv_rows(x, conv, state, out, _Rows(portion, slots))
@@ -472,7 +472,7 @@ def test_the_convolution_in_portions_and_token_by_token(taps, width):
     for s in range(2):
         state.zero_()
         w1 = P.input_convolution(unit[s].double().cpu().numpy(), conv.double().cpu().numpy().T)
-        for t in range(lengths[s]):
+        for t in range(40):
             out = torch.zeros((1, width), dtype=torch.float32, device="cuda:0")
             ops.sandwich_rows(base=unit[s][t:t + 1].contiguous(), out=out, norm_weight=ones, eps=0.0, conv=conv, state=state, batch=_Rows([1], [slots[s]]))
             assert np.abs(out.cpu().numpy()[0] - w1[t]).max() < 3e-5
@@ -611,6 +611,68 @@ def test_values_that_are_the_keys_in_the_cache(sizes, rows, dtype):
     at = lambda plane: np.stack([plane[perm[p // 64], :, p % 64] for p in pos])
     assert np.abs(at(kd) - turned(k)).max() < tol
     assert np.array_equal(at(vd), k)                        # as projected, bit for bit
+
+
+@pytest.mark.parametrize("shape", [(5, 70, 64, 96), (16, 700, 128, 256), (3, 300, 520, 40)])
+def test_squared_products_of_groups_in_one_launch(shape):
+    import torch
+    from gophonic_b200 import ops
+    ops.use_device(0)
+    groups, rows, K, N = shape
+    rng = np.random.default_rng(sum(shape))
+    sizes = rng.multinomial(rows, rng.dirichlet(np.ones(groups)))
+    sizes[0] += sizes[1]
+    sizes[1] = 0                                               # a group without rows
+    offsets = torch.tensor(np.concatenate([[0], np.cumsum(sizes)]), dtype=torch.int32, device="cuda:0")
+    a = torch.tensor(rng.standard_normal((rows, K)), dtype=torch.float32).bfloat16().cuda()
+    w = torch.tensor(rng.standard_normal((groups * N, K)) / np.sqrt(K), dtype=torch.float32).bfloat16().cuda()
+    out = torch.zeros((rows, N), dtype=torch.bfloat16, device="cuda:0")
+    ops.gemm_grouped(a, w, out, offsets, groups, gate="relu2")
+    torch.cuda.synchronize()
+    assert ops.tc5_status() == 0
+    z = np.concatenate([a.double().cpu().numpy()[o:o + n] @ w.double().cpu().numpy()[e * N:(e + 1) * N].T
+                        for e, (o, n) in enumerate(zip(offsets.tolist(), sizes))])
+    want = np.maximum(z, 0.0) ** 2
+    assert (np.abs(out.double().cpu().numpy() - want) / (1.0 + want)).max() < 1e-2
+
+
+@pytest.mark.parametrize("kind", ["relu2", "swiglu", "glu_clamp"])
+@pytest.mark.parametrize("shape", [(5, 3, 16, 64, 96), (8, 2, 9, 72, 24), (4, 4, 3, 2048, 128), (3, 1, 16, 40, 1536)])
+def test_few_rows_sorted_by_expert_on_the_tensor_cores(shape, kind):
+    """Experts with no pair, with a few and with more than one tile of pairs; inner sizes that are no multiple of a step."""
+    import torch
+    from gophonic_b200 import ops
+    ops.use_device(0)
+    E, top, rows, hidden, ff = shape
+    rng = np.random.default_rng(sum(shape))
+    per = 1 if kind == "relu2" else 2
+    as_bf = lambda a: torch.tensor(a, dtype=torch.float32).bfloat16().cuda()
+    x, up = as_bf(rng.standard_normal((rows, hidden))), as_bf(rng.standard_normal((E * per * ff, hidden)) / np.sqrt(hidden))
+    down = as_bf(rng.standard_normal((hidden, E * ff)) / np.sqrt(ff))
+    chosen = np.stack([np.sort(rng.permutation(E)[:top]) for _ in range(rows)])
+    chosen[:, 0] = 0 if E > top else chosen[:, 0]              # one expert takes every row
+    index = torch.tensor(chosen, dtype=torch.int32, device="cuda:0")
+    i32 = lambda n: torch.zeros(n, dtype=torch.int32, device="cuda:0")
+    offsets, place, src = i32(E + 1), i32(rows * top), i32(rows * top)
+    ops.moe_group(index, E, offsets, place, src)
+    ys = torch.zeros((rows * top, hidden), dtype=torch.float32, device="cuda:0")
+    ops.moe_rows_grouped(x, up, down, offsets, src, ys, E, top, ff, kind=kind, limit=1.0, slope=1.7)
+    torch.cuda.synchronize()
+    X, U, D = (t.double().cpu().numpy() for t in (x, up, down))
+    for r in range(rows):
+        for j in range(top):
+            e = chosen[r, j]
+            z = U[e * per * ff:(e + 1) * per * ff] @ X[r]
+            if kind == "relu2":
+                a = np.maximum(z, 0) ** 2
+            elif kind == "swiglu":
+                a = P.silu(z[:ff]) * z[ff:]
+            else:
+                c = np.minimum(z[:ff], 1.0)
+                a = c * P.sigmoid(1.7 * c) * (np.clip(z[ff:], -1.0, 1.0) + 1.0)
+            want = D[:, e * ff:(e + 1) * ff] @ a
+            got = ys[place[r * top + j].item()].double().cpu().numpy()
+            assert np.abs(got - want).max() < 4e-2 * max(1.0, np.abs(want).max())
 
 
 def test_capped_logits():

@@ -168,7 +168,7 @@ def test_the_cache_keeps_a_blocks_state_beside_its_mixers():
     with pytest.raises(CacheError, match="block"):
         Cache([reqs[0], (reqs[0][0], 0)], max_tokens=64, device="cpu", dtype=torch.float32)
     odd = ZenoraxConfig.from_dict(CONFIGS["odd"]).model_spec()          # one tap: nothing to keep
-    assert registry.part_class("block", "sandwich").cache_request(odd.layers[2]).shape == (1, 5)
+    assert registry.part_class("block", "sandwich").cache_request(odd.layers[2]).shape == (1, 15)
 
 
 def test_the_plain_convolution_and_average():
