@@ -231,7 +231,7 @@ __global__ void __launch_bounds__(256) conv_rows_kernel(const float* __restrict_
     const int seq = row_seq[row];
     const int local = (int)(row - seq_q_start[seq]);     // the row's place in its sequence's portion
     int slot = seq_slot[seq];
-    if (!gb_check(slot, max_slots, GB_CHECK_SLOT)) slot = 0;
+    if (taps > 1 && !gb_check(slot, max_slots, GB_CHECK_SLOT)) slot = 0;      // one tap reaches nothing back: there is no state
     const float* st = state + (int64_t)slot * state_slot_stride;
     for (int c = threadIdx.x * V; c < n; c += 256 * V) {
         float a[V], x[V], cw[V];

@@ -292,7 +292,14 @@ def random_weights(cfg: dict, seed: int, decided: bool = False) -> Dict[str, np.
         elif last == "sink":
             v = 1.0 + rng.standard_normal(shape)
         elif last == "correction":
-            v = 1.5 * (rng.permutation(shape[0]) - shape[0] // 2) if decided else 0.4 * rng.standard_normal(shape) - 0.5
+            if decided:      # whole groups one behind the other, so that their sums of two lie apart as well
+                router = cfg["layers"][int(name[1:name.index(".")])]["mlp"]["router"]
+                count = (router.get("groups") or {"count": 1})["count"]
+                per = shape[0] // count
+                ranks = np.concatenate([r * per + rng.permutation(per) for r in rng.permutation(count)])
+                v = 1.5 * (ranks - shape[0] // 2)
+            else:
+                v = 0.4 * rng.standard_normal(shape) - 0.5
         elif name == "embed":
             v = rng.standard_normal(shape)
         elif last == "router":

@@ -42,7 +42,7 @@ def test_the_spec_carries_the_designs_constants():
     assert spec.head.tied_to == "embed" and spec.head.soft_cap == 20.0 and spec.embedding.scale == 0.7
     assert [l.average for l in spec.layers] == [2, 3, 4, 5, 6, 7] and all(l.block == "sandwich" and l.conv_taps == 4 for l in spec.layers)
     a = spec.layers[0].mixer
-    assert a.kind == "gated_attention" and (a.heads, a.kv_heads, a.head_dim, a.value_dim, a.scale) == (4, 2, 16, 16, 0.5)
+    assert a.kind == "gated_attention" and (a.heads, a.kv_heads, a.head_dim, a.value_dim, a.scale) == (4, 2, 16, 16, 0.3)
     assert a.value_from_key and a.sink_learned and not a.qk_norm_weight and a.qk_norm_after and a.qk_norm.eps == 1e-5 and a.window == 0
     assert a.position.kind == "rope" and (a.position.rotary_dim, a.position.theta, a.position.scaling) == (8, 100.0, LinearStretch(2.5))
     h = spec.layers[1].mixer
