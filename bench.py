@@ -284,16 +284,17 @@ def further_model_points(name, steps, torch, ops, hbm_peak, tflops_peak):
 # both mix matrix-state layers with windowed attention; a Kalonex configuration, all attention and gated feed-forwards,
 # beside the Qwen3-shaped one of its width; a Kimilix configuration, windowed attention and mixtures with a shared expert,
 # beside the Kalonex one of its width; a Zenorax configuration, latent attention and mixtures that read as many expert rows
-# a token, beside the Kimilix one of its width)
+# a token, beside the Kimilix one of its width; a Lefalix configuration, delta rules and windowed attention behind short
+# convolutions, beside the Vepitar one of its width)
 DESIGN_TWINS = {"pugalix-2k": "1.7b", "pugalix-4k": "8b", "vepitar-2k": "pugalix-2k", "vepitar-4k": "pugalix-4k",
                 "kalonex-2k": "1.7b", "kalonex-4k": "8b", "kimilix-2k": "kalonex-2k", "kimilix-4k": "kalonex-4k",
-                "zenorax-2k": "kimilix-2k", "zenorax-4k": "kimilix-4k"}
+                "zenorax-2k": "kimilix-2k", "zenorax-4k": "kimilix-4k", "lefalix-2k": "vepitar-2k", "lefalix-4k": "vepitar-4k"}
 OP_CLASSES = ("gemm", "gemm_add", "gemm_swiglu", "gemm_scaled", "gemm_residual", "attention", "attention_decode_rope",
               "qk_norm_rope_kv_write", "state_scan", "head_norm_gate", "gla_decay", "add_rmsnorm", "embed_gather", "swiglu",
               "prenorm_layer_forward", "embed_streams", "delta_scan", "conv_qkv", "attention_sigmoid", "hyper_mix_norm", "moe_route", "moe_act", "moe_rows",
               "moe_rows_grouped", "moe_group", "moe_gather", "moe_combine", "relu2", "tanh_", "add_bias", "concat_cast", "add_rows", "gemm_w_cols", "gemm_grouped",
               "norm_scale_add", "diff_combine", "add_rows_gated", "latent_prep", "latent_q_rot", "head_gemm", "head_gemm_mma", "f32_to_bf16",
-              "sandwich_rows", "conv_rows", "soft_cap_")
+              "sandwich_rows", "conv_rows", "soft_cap_", "short_conv", "gated_delta", "gelu")
 
 
 class OpTimer:

@@ -36,7 +36,7 @@ from typing import Dict, List, Optional, Sequence, Tuple
 import numpy as np
 import torch
 
-from ..parts.base import BlockStateRequest, KVRequest, KVStateRequest, StateRequest
+from ..parts.base import BlockStateRequest, KVRequest, KVStateRequest, PartsRequest, StateRequest
 
 PAGE = 64
 
@@ -123,6 +123,13 @@ class BlockView:
 
 
 @dataclass
+class PartsView:
+    """The view of a run whose mixer asked for several pieces: the pieces' views, in order."""
+    parts: Tuple[object, ...]
+    writable: bool = True
+
+
+@dataclass
 class CacheMark:
     """What ``Cache.snapshot`` returns: a length and the state of that moment."""
     slot: int
@@ -161,6 +168,7 @@ class Cache:
         self._plane: Dict[int, Tuple[str, object, int]] = {}
         self._beside: Dict[int, Tuple[object, int]] = {}     # the state plane of a run that asked for keys and state
         self._of_block: Dict[int, Tuple[object, int]] = {}   # the state plane of a run whose block asked for one
+        self._pieces: Dict[object, List[object]] = {}        # the pieces of a run (or piece) that asked for several
         self._cache_of: Dict[int, Optional[int]] = {}
         for pos, (req, cache_of) in enumerate(requests):
             self._cache_of[pos] = cache_of
@@ -172,35 +180,11 @@ class Cache:
                 self._of_block[pos] = (key, len(planes))
                 planes.append(pos)
                 req = req.mixer
-            if cache_of is not None or req is None:
+            if isinstance(req, PartsRequest) and cache_of is not None:
+                raise CacheError(f"schedule position {pos}: a run whose mixer has several pieces cannot read another run's cache")
+            if cache_of is not None:
                 continue
-            if isinstance(req, KVStateRequest):
-                key = (tuple(req.state.shape), req.state.dtype)
-                planes = self._state_groups.setdefault(key, [])
-                self._beside[pos] = (key, len(planes))
-                planes.append(pos)
-                req = req.kv
-            if isinstance(req, KVRequest):
-                # values as wide as keys: the key every such group has always had; else the width is part of it
-                key = (req.kv_heads, req.head_dim, req.window)
-                vheads, in_keys = int(getattr(req, "value_heads", 0) or 0), bool(getattr(req, "values_in_keys", False))
-                if (vheads and vheads != req.kv_heads) or in_keys:
-                    # value heads of their own count, or values that are channels of the keys: the whole geometry is the key
-                    if in_keys and (vheads not in (0, req.kv_heads) or (req.value_dim or req.head_dim) > req.head_dim):
-                        raise CacheError(f"schedule position {pos}: values inside the keys need as many value heads, no wider than the keys")
-                    key += (req.value_dim or req.head_dim, vheads or req.kv_heads, in_keys)
-                elif req.value_dim and req.value_dim != req.head_dim:
-                    key += (req.value_dim,)
-                planes = self._kv_groups.setdefault(key, [])
-                self._plane[pos] = ("kv", key, len(planes))
-                planes.append(pos)
-            elif isinstance(req, StateRequest):
-                key = (tuple(req.shape), req.dtype)
-                planes = self._state_groups.setdefault(key, [])
-                self._plane[pos] = ("state", key, len(planes))
-                planes.append(pos)
-            else:
-                raise CacheError(f"schedule position {pos}: unknown cache request {req!r}")
+            self._place(pos, req)
         for pos, cache_of in self._cache_of.items():
             if cache_of is not None and cache_of not in self._plane:
                 raise CacheError(f"schedule position {pos} reads the cache of position {cache_of}, which has none")
@@ -219,6 +203,44 @@ class Cache:
             self._state[key] = torch.zeros((len(planes), self.max_slots + 1) + tuple(shape), dtype=sdtype, device=self.device)
         self._ops = None
         self._stager = None
+
+    def _place(self, pos, req) -> None:
+        """Give a run (``pos`` its schedule position) or one piece of it (``pos`` the pair of what it belongs to and its number)
+        its planes."""
+        if req is None:
+            return
+        if isinstance(req, PartsRequest):
+            self._pieces[pos] = [(pos, i) for i in range(len(req.parts))]
+            for at, piece in zip(self._pieces[pos], req.parts):
+                self._place(at, piece)
+            return
+        if isinstance(req, KVStateRequest):
+            key = (tuple(req.state.shape), req.state.dtype)
+            planes = self._state_groups.setdefault(key, [])
+            self._beside[pos] = (key, len(planes))
+            planes.append(pos)
+            req = req.kv
+        if isinstance(req, KVRequest):
+            # values as wide as keys: the key every such group has always had; else the width is part of it
+            key = (req.kv_heads, req.head_dim, req.window)
+            vheads, in_keys = int(getattr(req, "value_heads", 0) or 0), bool(getattr(req, "values_in_keys", False))
+            if (vheads and vheads != req.kv_heads) or in_keys:
+                # value heads of their own count, or values that are channels of the keys: the whole geometry is the key
+                if in_keys and (vheads not in (0, req.kv_heads) or (req.value_dim or req.head_dim) > req.head_dim):
+                    raise CacheError(f"schedule position {pos}: values inside the keys need as many value heads, no wider than the keys")
+                key += (req.value_dim or req.head_dim, vheads or req.kv_heads, in_keys)
+            elif req.value_dim and req.value_dim != req.head_dim:
+                key += (req.value_dim,)
+            planes = self._kv_groups.setdefault(key, [])
+            self._plane[pos] = ("kv", key, len(planes))
+            planes.append(pos)
+        elif isinstance(req, StateRequest):
+            key = (tuple(req.shape), req.dtype)
+            planes = self._state_groups.setdefault(key, [])
+            self._plane[pos] = ("state", key, len(planes))
+            planes.append(pos)
+        else:
+            raise CacheError(f"schedule position {pos}: unknown cache request {req!r}")
 
     @staticmethod
     def _geometry(key) -> Tuple[int, int, int, int, int, bool]:
@@ -256,6 +278,8 @@ class Cache:
         return self._mixer_view(pos)
 
     def _mixer_view(self, pos: int):
+        if pos in self._pieces:
+            return PartsView(tuple(self._mixer_view(at) for at in self._pieces[pos]))
         src = self._cache_of.get(pos)
         writable = src is None
         at = pos if src is None else src

@@ -1,5 +1,6 @@
 from .spec import ClampedGLUSpec, DiffAttentionSpec, LatentAttentionSpec, PostNormLayerSpec, ReluSquaredSpec
 from .spec import ForgetStateSpec, LinearStretch, RampStretch, SandwichLayerSpec
+from .spec import AddStartSpec, GatedDeltaSpec, GeluSpec, ParallelSpec
 from .spec import (AttentionSpec, DecayStateSpec, DeltaRuleSpec, EmbeddingSpec, GatedAttentionSpec, HeadSpec, HyperLayerSpec,
                    LayerSpec, MatrixMemorySpec, MoESpec, ModelSpec, NoPositionSpec, PairRotarySpec, RMSNormSpec, ReinjectSpec, RotarySpec,
                    ScheduleEntry, SigmoidAttentionSpec, SwiGLUSpec, default_schedule)
@@ -9,10 +10,11 @@ from .vepitar import VepitarConfig
 from .kalonex import KalonexConfig
 from .kimilix import KimilixConfig
 from .zenorax import ZenoraxConfig
+from .lefalix import LefalixConfig
 
 __all__ = ["AttentionSpec", "DecayStateSpec", "DeltaRuleSpec", "EmbeddingSpec", "GatedAttentionSpec", "HeadSpec", "HyperLayerSpec",
            "LayerSpec", "MatrixMemorySpec", "MoESpec", "ModelSpec", "NoPositionSpec", "PairRotarySpec", "RMSNormSpec", "ReinjectSpec", "RotarySpec",
            "ScheduleEntry", "SigmoidAttentionSpec", "SwiGLUSpec", "default_schedule", "ConfigError", "Qwen3Config", "PugalixConfig",
            "VepitarConfig", "KalonexConfig", "KimilixConfig", "ClampedGLUSpec", "DiffAttentionSpec", "LatentAttentionSpec",
            "PostNormLayerSpec", "ReluSquaredSpec", "ForgetStateSpec", "LinearStretch", "RampStretch", "SandwichLayerSpec",
-           "ZenoraxConfig"]
+           "ZenoraxConfig", "AddStartSpec", "GatedDeltaSpec", "GeluSpec", "ParallelSpec", "LefalixConfig"]

@@ -121,8 +121,11 @@ class GatedAttentionSpec:
       position encoding; with ``qk_norm_span`` over the whole projection at once (all heads of q share one mean of
       squares and a weight of heads * head_dim, tensor ``q.norm``; k likewise), else head by head with a weight
       of head_dim.  ``qk_norm_weight`` False: a norm without a weight (no tensors); ``qk_norm_after``: the norm stands
-      behind the position encoding (only without a weight, and with an encoding that keeps a head's length: then the
-      two orders are the same function, since a rotation changes no sum of squares);
+      behind the position encoding (only without a weight; with an encoding that keeps a head's length the two orders are
+      the same function, since a rotation changes no sum of squares);
+    * ``conv_taps`` > 0: a causal convolution over time on every channel of q, k and v directly behind the projection and its
+      bias, y_t = sum_j c[:, j] u_(t - taps + 1 + j), zeros before the sequence's start (tensors: the projection's name plus
+      ``conv_suffix``, [channels, taps]); a sequence's last taps - 1 projected rows are part of its state;
     * ``value_from_key``: there is no value projection, the values are the keys as projected, before norm and rotation
       (``value_dim`` = ``head_dim``);
     * ``out_bias``: the output projection carries a bias too;
@@ -153,9 +156,11 @@ class GatedAttentionSpec:
     qk_norm_weight: bool = True
     qk_norm_after: bool = False
     value_from_key: bool = False
+    conv_taps: int = 0
     names: Tuple[Tuple[str, str], ...] = (("q", "q"), ("k", "k"), ("v", "v"), ("g", "g"), ("o", "o"), ("q_norm", "q.norm"),
                                           ("k_norm", "k.norm"), ("sink", "sink"))
     bias_suffix: str = ".b"
+    conv_suffix: str = ".conv"
     kind: str = "gated_attention"
 
 
@@ -277,6 +282,52 @@ class DeltaRuleSpec:
 
 
 @dataclass(frozen=True)
+class GatedDeltaSpec:
+    """The gated delta rule: per head a matrix state S (key_dim x value_dim, float32) with a decay g and a write strength b,
+
+        S <- diag(g) S,   u = b (v - S^T k),   S <- S + k u^T,   o = S^T q      (the read-out sees the token's own write).
+
+    q and k have ``kv_heads`` heads of key_dim (head h reads head h // (heads / kv_heads)), v ``heads`` of value_dim.  Each passes
+    a short causal convolution over time per channel (``conv_taps``; 0: none; tensors: the projection's name plus ``conv_suffix``)
+    and silu; q and k are then unit vectors per head, x / sqrt(sum(x^2) + unit_eps), and q is scaled by key_dim^(-1/2).
+    b = sigmoid(W_b x) per head.  The decay is g = exp(-exp(A_h) softplus(z + dt_bias)), with z one number per head, W_a x, or with
+    ``channel_decay`` one per head and key channel, W_a2 (W_a1 x), W_a1 of ``rank`` rows (None: the checkpoint's).
+    Each head's o is divided by its root mean square (``eps``), multiplied by a weight of value_dim shared by the heads and by
+    ``gate`` ("silu" or "sigmoid") of W_g x or, with ``gate_low_rank``, of W_g2 (W_g1 x), W_g1 of ``gate_rank`` rows, and projected back."""
+    hidden: int
+    heads: int
+    kv_heads: int
+    key_dim: int
+    value_dim: int
+    eps: float
+    conv_taps: int = 0
+    unit_eps: float = 1e-6
+    channel_decay: bool = False
+    rank: Optional[int] = None
+    gate: str = "silu"
+    gate_low_rank: bool = False
+    gate_rank: Optional[int] = None
+    names: Tuple[Tuple[str, str], ...] = (("q", "q"), ("k", "k"), ("v", "v"), ("b", "b"), ("a", "a"), ("a1", "a1"), ("a2", "a2"),
+                                          ("a_log", "A_log"), ("dt_bias", "dt_bias"), ("norm", "norm"), ("g", "g"), ("g1", "g1"), ("g2", "g2"),
+                                          ("o", "o"))
+    conv_suffix: str = ".conv"
+    kind: str = "gated_delta"
+
+
+@dataclass(frozen=True)
+class ParallelSpec:
+    """Two mixers side by side that read the same input, their tensors under ``prefixes``; the result is the sum of their outputs,
+    each RMS-normed over the model width (``eps``) with a weight of its own (tensors ``prefixes[i] + out_name``), times ``factor``."""
+    hidden: int
+    mixers: Tuple[object, object]
+    eps: float
+    factor: float = 0.5
+    prefixes: Tuple[str, str] = ("left.", "right.")
+    out_name: str = "out"
+    kind: str = "parallel"
+
+
+@dataclass(frozen=True)
 class ForgetStateSpec:
     """HGRN2: linear attention whose forget gate also decides what is written.  Per head a matrix state S (key_dim x
     value_dim, float32), with q = silu(W_q x), v = W_v x and per key channel
@@ -347,7 +398,7 @@ class MoESpec:
     * ``correction``: an expert is chosen by its score plus a learned number (tensor ``correction_name``, one an expert);
       the weights come from the score without it;
     * ``groups`` > 1: the experts form that many equal groups of neighbours, a group counts as the sum of its two largest
-      choice scores, and only experts of the ``keep_groups`` best groups can be chosen."""
+      choice scores, or with ``group_rank`` "largest" as its largest, and only experts of the ``keep_groups`` best groups can be chosen."""
     hidden: int
     experts: int
     top: int
@@ -370,6 +421,7 @@ class MoESpec:
     correction_name: str = "correction"
     groups: int = 1
     keep_groups: int = 1
+    group_rank: str = "two_largest"
 
 
 @dataclass(frozen=True)
@@ -388,6 +440,16 @@ class ReluSquaredSpec:
     hidden: int
     intermediate: int
     kind: str = "relu2_ff"
+    names: Tuple[str, str] = ("up", "down")
+
+
+@dataclass(frozen=True)
+class GeluSpec:
+    """down(gelu(up(x))), gelu(z) = z times the normal law's distribution function at z.  ``names``: the tensors of the up and down
+    projections under the part's prefix."""
+    hidden: int
+    intermediate: int
+    kind: str = "gelu_ff"
     names: Tuple[str, str] = ("up", "down")
 
 
@@ -526,6 +588,13 @@ class ReinjectSpec:
 
 
 @dataclass(frozen=True)
+class AddStartSpec:
+    """What happens to the residual where a pass through repeated layers begins: x <- x + x0, x0 the embedding output."""
+    hidden: int
+    kind: str = "add_start"
+
+
+@dataclass(frozen=True)
 class ScheduleEntry:
     """One run of a layer.
 
@@ -533,7 +602,7 @@ class ScheduleEntry:
     then used more than once, each run with a cache plane of its own).  ``cache_of`` names the
     schedule position whose cache plane this run reads instead of writing one of its own
     (None: own plane).  ``enter``: the spec of a *junction* part (registry category ``junction``) that
-    rewrites the residual right before this run (``ReinjectSpec``), or None.
+    rewrites the residual right before this run (``ReinjectSpec``, ``AddStartSpec``), or None.
     """
     layer: int
     cache_of: Optional[int] = None

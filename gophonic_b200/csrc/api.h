@@ -309,7 +309,8 @@ struct MoeRouteParams {
     int renorm;             // 1: the chosen scores are divided by their sum + renorm_eps; 0: they are the weights
     const float* correction;   // [experts] added to the scores for the choice alone, or null
     int groups, keep_groups;   // groups > 1: equal groups of neighbours; only experts of the keep_groups best ones (sum of a group's
-                               // two largest choice scores) can be chosen
+                               // two largest choice scores, or the largest alone) can be chosen
+    int group_largest;         // 1: a group counts as its largest choice score
 };
 GB_API int gb_moe_route(const MoeRouteParams* p, cudaStream_t stream);
 GB_API int gb_moe_act(const void* up, int64_t up_stride, const float* dense, void* act, int64_t act_stride, int rows, int experts, int ff,
@@ -386,9 +387,74 @@ struct SandwichParams {
     const int* seq_slot;
     int max_slots;
     int rows, width;
+    const float* y2;        // a second output beside y, or null; with it y / rms(y) * pair_w + y2 / rms(y2) * pair_w2 stands for y
+    const float* pair_w;
+    const float* pair_w2;
+    float pair_eps;
 };
 GB_API int gb_sandwich_rows(const SandwichParams* p, int out_dtype, cudaStream_t stream);
 GB_API int gb_conv_rows(const float* h, const float* conv_w, int taps, float* state, int64_t state_slot_stride, int max_slots, void* out, int out_dtype,
                         int rows, int width, int nseq, const int* row_seq, const int* seq_slot, const int* seq_q_start, const int* seq_q_len,
                         cudaStream_t stream);
 GB_API int gb_soft_cap(float* z, int64_t n, float cap, cudaStream_t stream);
+
+// The short convolution on projected heads with what follows it up to the mixer's arithmetic (short_conv.cu).
+struct ShortConvParams {
+    const void* src;        // [rows, row_stride]: q heads, k heads (d wide), v heads (dv wide), then anything else
+    int64_t row_stride;
+    const float* conv_w;    // [taps][channels], the last row the current token's, or null with taps 1
+    const float* bias;      // [channels] of the projection, or null
+    int taps, channels;
+    float* state;           // [slots, state_slot_stride]: the last taps - 1 projected rows with their bias, oldest first
+    int64_t state_slot_stride;
+    int silu;               // 1: silu behind the convolution
+    int norm;               // q and k heads, behind the rotation: 0 none, 1 x / sqrt(mean x^2 + eps), 2 x / sqrt(sum x^2 + eps)
+    float eps, q_scale;
+    const float* cos_t;     // [table_positions, rot / 2]
+    const float* sin_t;
+    int rot, pairs, table_positions;
+    int to_cache;           // 1: out receives the q heads alone, in the activation dtype, k and v go to the cache; 0: out receives all
+    void* out;              // channels as float32
+    int64_t out_stride;
+    const int* block_table;
+    int bt_stride, pages;
+    void* k_plane;
+    void* v_plane;
+    const int* row_pos;
+    const int* row_seq;
+    const int* seq_slot;
+    const int* seq_q_start;
+    const int* seq_q_len;
+    int rows, nseq, q_heads, k_heads, v_heads, d, dv;
+    int max_slots, max_q_len;
+    int vec;                // set by the library
+};
+GB_API int gb_short_conv(const ShortConvParams* p, int dtype, cudaStream_t stream);
+
+// The gated delta rule (gated_delta.cu).
+struct GatedDeltaParams {
+    const float* rows_in;   // [rows, row_stride]: unit q (scaled) and k heads, d wide, kv_heads each, and v heads, dv wide
+    int64_t row_stride;
+    int q_off, k_off, v_off;
+    const float* decay_in;  // pre-activations [rows, decay_stride]: one a head, or (per_channel) one a head and key channel
+    int64_t decay_stride;
+    const float* dt_bias;   // [heads] or [heads * d]
+    const float* a_log;     // [heads]
+    const float* beta_in;   // [rows, beta_stride]: pre-activations, one a head
+    int64_t beta_stride;
+    float* decay_out;       // [rows, heads (* d)] scratch: the factors; not used for single tokens
+    float* coef;            // [rows, heads, 8] scratch; not used for single tokens
+    float* state;           // [slots, slot_stride], a head's matrix [d][dv] at head_stride
+    int64_t slot_stride, head_stride;
+    float* out;             // [rows, out_stride]
+    int64_t out_stride;
+    const int* row_seq;
+    const int* seq_slot;
+    const int* seq_q_start;
+    const int* seq_q_len;
+    int rows, nseq, heads, kv_heads, d, dv;
+    int per_channel, max_slots, max_q_len;
+    int narrow_below;       // with fewer (head, 16 columns) pairs than this a warp takes two columns instead of four
+};
+GB_API int gb_gated_delta(const GatedDeltaParams* p, cudaStream_t stream);
+GB_API int gb_gelu(void* z, int64_t n, int dtype, cudaStream_t stream);

@@ -55,6 +55,8 @@ SOURCES = [
     "postnorm.cu",
     "attention_latent.cu",
     "sandwich.cu",
+    "short_conv.cu",
+    "gated_delta.cu",
     "sampling.cu",
     "no_alloc.cu",
     "dispatch.cu",

@@ -7,7 +7,7 @@
 // that reads only the chosen experts' matrices.
 //
 // With a correction an expert is chosen by its score plus a learned number and weighed by the score; with groups only
-// experts of the best groups of neighbours (by the sum of a group's two largest choice scores) can be chosen.
+// experts of the best groups of neighbours (by the sum of a group's two largest choice scores, or by its largest) can be chosen.
 //
 // moe_act: act[r, e * ff + i] = weight[r, e] * relu(up[r, e * ff + i])^2: the activation of every expert's
 // hidden layer with the row's weight for that expert folded in, so that one product with the experts' down
@@ -36,9 +36,9 @@ namespace {
 constexpr int MAX_EXPERTS_PER_LANE = 16;   // experts up to 512
 
 // Which experts may be chosen: with groups, `key` (the warp's choice scores in shared memory) is scanned by a lane a group
-// for the group's two largest, and a group is kept if fewer than keep_groups groups come before it (a larger sum, or an
+// for the group's two largest (which count together, or with `largest` the first alone), and a group is kept if fewer than keep_groups groups come before it (a larger sum, or an
 // equal one and a lower number).  Scores of the other groups become -inf.
-__device__ __forceinline__ void drop_groups(float* key, float* strength, int E, int groups, int keep, int lane) {
+__device__ __forceinline__ void drop_groups(float* key, float* strength, int E, int groups, int keep, int largest, int lane) {
     const int per = E / groups;
     for (int g = lane; g < groups; g += 32) {
         float a = -INFINITY, b = -INFINITY;
@@ -51,7 +51,7 @@ __device__ __forceinline__ void drop_groups(float* key, float* strength, int E, 
                 b = v;
             }
         }
-        strength[g] = per > 1 ? a + b : a;
+        strength[g] = per > 1 && !largest ? a + b : a;
     }
     __syncwarp();
     for (int g = lane; g < groups; g += 32) {
@@ -105,7 +105,7 @@ __global__ void __launch_bounds__(128) moe_route_kernel(MoeRouteParams p) {
         }
         if (p.groups > 1) {
             __syncwarp();
-            drop_groups(key_s[warp], group_s[warp], E, p.groups, p.keep_groups, lane);
+            drop_groups(key_s[warp], group_s[warp], E, p.groups, p.keep_groups, p.group_largest, lane);
 #pragma unroll
             for (int e = 0; e < MAX_EXPERTS_PER_LANE; e++)
                 if (lane + 32 * e < E) s[e] = key_s[warp][lane + 32 * e];
@@ -465,6 +465,27 @@ __global__ void moe_gather_kernel(const T* __restrict__ x, int64_t x_stride, con
     }
 }
 
+// z times the normal law's distribution function at z
+__device__ __forceinline__ float gelu_erf(float z) { return 0.5f * z * (1.f + erff(z * 0.70710678118654752f)); }
+
+// V elements a thread: 16 bytes where rows allow it
+template <typename T, int V>
+__global__ void gelu_kernel(T* __restrict__ z, int64_t n) {
+    pdl_wait();
+    pdl_trigger();
+    const int64_t i = ((int64_t)blockIdx.x * blockDim.x + threadIdx.x) * V;
+    if (i >= n) return;
+    if constexpr (V > 1) {
+        uint4 raw = *reinterpret_cast<const uint4*>(z + i);
+        T* t = reinterpret_cast<T*>(&raw);
+#pragma unroll
+        for (int u = 0; u < V; u++) t[u] = from_f32<T>(gelu_erf(to_f32<T>(t[u])));
+        *reinterpret_cast<uint4*>(z + i) = raw;
+    } else {
+        z[i] = from_f32<T>(gelu_erf(to_f32<T>(z[i])));
+    }
+}
+
 template <typename T>
 __global__ void relu2_kernel(T* __restrict__ z, int64_t n) {
     const int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x;
@@ -523,6 +544,26 @@ GB_API int gb_relu2(void* z, int64_t n, int dtype, cudaStream_t stream) {
     else
         GB_REFUSE("relu2: unknown dtype %d", dtype);
     GB_CHECK_LAUNCH("relu2");
+    return 0;
+}
+
+GB_API int gb_gelu(void* z, int64_t n, int dtype, cudaStream_t stream) {
+    if (n <= 0) return 0;
+    const int v = dtype == GB_BF16 ? 8 : 4;
+    const bool vec = !(n % v) && !((uintptr_t)z & 15);
+    const int64_t threads = vec ? n / v : n, blocks = (threads + 255) / 256;
+    if (blocks > 0x7fffffff) GB_REFUSE("gelu: %lld elements are too many for one launch", (long long)n);
+    const dim3 grid((unsigned)blocks), block(256);
+    if (dtype == GB_F32) {
+        if (vec) launch_pdl(gelu_kernel<float, 4>, grid, block, 0, stream, (float*)z, n);
+        else launch_pdl(gelu_kernel<float, 1>, grid, block, 0, stream, (float*)z, n);
+    } else if (dtype == GB_BF16) {
+        if (vec) launch_pdl(gelu_kernel<__nv_bfloat16, 8>, grid, block, 0, stream, (__nv_bfloat16*)z, n);
+        else launch_pdl(gelu_kernel<__nv_bfloat16, 1>, grid, block, 0, stream, (__nv_bfloat16*)z, n);
+    } else {
+        GB_REFUSE("gelu: unknown dtype %d", dtype);
+    }
+    GB_CHECK_LAUNCH("gelu");
     return 0;
 }
 

@@ -1,7 +1,8 @@
 // Row-wise kernels of blocks that norm in front of and behind their sublayers, convolve what a mixer reads over a few
 // tokens and weigh the results of all layers so far into what goes on; and the cap on a head's logits.
 //
-// sandwich_rows:  between two sublayers, one pass over a row of the float32 residual: the sublayer's output over its root
+// sandwich_rows:  between two sublayers, one pass over a row of the float32 residual: the sublayer's output (or the sum of two
+//                 outputs side by side, each over its own root mean square and times a weight) over its root
 //                 mean square and times its weight joins the residual (the sum may be stored: a layer's result), the planes
 //                 of the earlier results and this one are summed with one weight each (stored if asked), and the sum is
 //                 normed for whoever reads it next.  For single tokens the normed row also passes the convolution, whose
@@ -33,6 +34,18 @@ __device__ __forceinline__ float block_sum(float v, float* part) {
     return t;
 }
 
+// the same for two values at once
+template <int THREADS>
+__device__ __forceinline__ void block_sum2(float& a, float& b, float* part_a, float* part_b) {
+    a = warp_sum(a);
+    b = warp_sum(b);
+    if ((threadIdx.x & 31) == 0) part_a[threadIdx.x >> 5] = a, part_b[threadIdx.x >> 5] = b;
+    __syncthreads();
+    a = b = 0.f;
+#pragma unroll
+    for (int i = 0; i < THREADS / 32; i++) a += part_a[i], b += part_b[i];
+}
+
 template <int V>
 __device__ __forceinline__ void load_v(const float* __restrict__ src, float* v) {
     if (V == 4) {
@@ -62,12 +75,12 @@ __device__ __forceinline__ void store_v(__nv_bfloat16* dst, const float* v) {
     }
 }
 
-// V neighbouring elements a piece, P pieces a thread, V * THREADS elements apart
-template <typename TO, int V, int P, int THREADS>
+// V neighbouring elements a piece, P pieces a thread, V * THREADS elements apart.  PAIR: the sublayer left two outputs, y and y2
+template <typename TO, int V, int P, int THREADS, bool PAIR>
 __global__ void __launch_bounds__(THREADS) sandwich_rows_kernel(SandwichParams p) {
     pdl_wait();
     pdl_trigger();
-    __shared__ float part[2][THREADS / 32];
+    __shared__ float part[PAIR ? 4 : 2][THREADS / 32];
     const int n = p.width;
     const int64_t out_row = blockIdx.x;
     const int64_t row = p.row_index ? p.row_index[out_row] : out_row;
@@ -127,6 +140,35 @@ __global__ void __launch_bounds__(THREADS) sandwich_rows_kernel(SandwichParams p
             if (c < n) load_v<V>(p.y + row * n + c, y[k]);
 #pragma unroll
             for (int u = 0; u < V; u++) ss += y[k][u] * y[k][u];
+        }
+        if (PAIR) {
+            float y2[P][V];
+            float s2 = 0.f;
+#pragma unroll
+            for (int k = 0; k < P; k++) {
+#pragma unroll
+                for (int u = 0; u < V; u++) y2[k][u] = 0.f;
+                const int c = c0 + k * STEP;
+                if (c < n) load_v<V>(p.y2 + row * n + c, y2[k]);
+#pragma unroll
+                for (int u = 0; u < V; u++) s2 += y2[k][u] * y2[k][u];
+            }
+            block_sum2<THREADS>(ss, s2, part[PAIR ? 2 : 0], part[PAIR ? 3 : 0]);
+            const float i1 = 1.0f / sqrtf(ss / (float)n + p.pair_eps), i2 = 1.0f / sqrtf(s2 / (float)n + p.pair_eps);
+            ss = 0.f;
+#pragma unroll
+            for (int k = 0; k < P; k++) {
+                const int c = c0 + k * STEP;
+                if (c >= n) continue;
+                float w1[V], w2[V];
+                load_v<V>(p.pair_w + c, w1);
+                load_v<V>(p.pair_w2 + c, w2);
+#pragma unroll
+                for (int u = 0; u < V; u++) {
+                    y[k][u] = fmaf(y[k][u] * i1, w1[u], y2[k][u] * i2 * w2[u]);
+                    ss += y[k][u] * y[k][u];
+                }
+            }
         }
         const float inv = 1.0f / sqrtf(block_sum<THREADS>(ss, part[0]) / (float)n + p.y_eps);
 #pragma unroll
@@ -191,7 +233,10 @@ __global__ void __launch_bounds__(THREADS) sandwich_rows_kernel(SandwichParams p
 
 template <typename TO, int V, int P, int THREADS>
 int launch_rows(const SandwichParams& p, cudaStream_t stream) {
-    launch_pdl(sandwich_rows_kernel<TO, V, P, THREADS>, dim3(p.rows), dim3(THREADS), 0, stream, p);
+    if (p.y2)
+        launch_pdl(sandwich_rows_kernel<TO, V, P, THREADS, true>, dim3(p.rows), dim3(THREADS), 0, stream, p);
+    else
+        launch_pdl(sandwich_rows_kernel<TO, V, P, THREADS, false>, dim3(p.rows), dim3(THREADS), 0, stream, p);
     GB_CHECK_LAUNCH("sandwich_rows");
     return 0;
 }
@@ -202,7 +247,8 @@ template <typename TO>
 int dispatch_rows(const SandwichParams& p, cudaStream_t stream) {
     const int n = p.width;
     const uintptr_t all = (uintptr_t)p.base | (uintptr_t)p.y | (uintptr_t)p.y_w | (uintptr_t)p.result | (uintptr_t)p.planes | (uintptr_t)p.x_out |
-                          (uintptr_t)p.norm_w | (uintptr_t)p.out | (uintptr_t)p.conv_w | (uintptr_t)p.state;
+                          (uintptr_t)p.norm_w | (uintptr_t)p.out | (uintptr_t)p.conv_w | (uintptr_t)p.state |
+                          (uintptr_t)p.y2 | (uintptr_t)p.pair_w | (uintptr_t)p.pair_w2;
     if (!(n & 3) && !(all & 15) && !(p.plane_stride & 3) && !(p.state_slot_stride & 3)) {
         if (p.rows < MANY_ROWS && n > 1024) {
             if (n <= 2048) return launch_rows<TO, 4, 1, 512>(p, stream);
@@ -334,6 +380,7 @@ GB_API int gb_sandwich_rows(const SandwichParams* pp, int out_dtype, cudaStream_
     if (p.rows <= 0) return 0;
     if (p.width <= 0 || p.n_planes < 0) GB_REFUSE("sandwich_rows: rows of %d, %d planes", p.width, p.n_planes);
     if (!p.base || !p.out || !p.norm_w || (p.y && !p.y_w) || (p.average && p.n_planes > 0 && !p.planes)) GB_REFUSE("sandwich_rows: a tensor is missing");
+    if (p.y2 && (!p.y || !p.pair_w || !p.pair_w2)) GB_REFUSE("sandwich_rows: two outputs side by side need both and their weights");
     if (p.row_index && (p.result || p.x_out || p.conv_w)) GB_REFUSE("sandwich_rows: gathered rows are only read");
     if (p.conv_w && (p.taps <= 0 || p.taps > MAX_TAPS)) GB_REFUSE("sandwich_rows: %d taps; 1 to %d", p.taps, MAX_TAPS);
     if (p.conv_w && (!p.row_seq || !p.seq_slot || (p.taps > 1 && (!p.state || p.state_slot_stride < (int64_t)(p.taps - 1) * p.width))))

@@ -65,8 +65,10 @@ class Model:
         # junctions: parts that rewrite the residual right before a run of the schedule
         self.junctions = {pos: registry.part_class("junction", e.enter.kind)(e.enter, "", tensors, runtime)
                           for pos, e in enumerate(spec.schedule) if getattr(e, "enter", None) is not None}
-        if self.junctions and (self._takes_streams[0] or self._takes_history[0]):
-            raise ValueError("model spec: a junction rewrites one residual; blocks that keep it in streams or planes cannot have one")
+        if self.junctions and self._takes_streams[0]:
+            raise ValueError("model spec: a junction rewrites one residual; blocks that keep it in streams cannot have one")
+        if self._takes_history[0] and not all(hasattr(j, "over_planes") for j in self.junctions.values()):
+            raise ValueError("model spec: ahead of blocks that read earlier layers' results a junction is a weighted sum of them")
         # a block arrangement may take the norm that follows it (to prepare the residual's rows for it)
         self._takes_next_norm = ["next_norm" in inspect.signature(b.forward).parameters for b in self.blocks]
         norm_prefix = final_norm_prefix(spec)
@@ -216,11 +218,14 @@ class Model:
         output, run i leaves plane i + 1, and what the last block leaves unfinished is completed for the wanted rows alone."""
         ops = self.rt.ops
         schedule = self.spec.schedule
-        planes = torch.empty((len(schedule) + 1, batch.rows, self.spec.hidden), dtype=torch.float32, device=self.rt.device)
+        # blocks that read nothing but the latest result and the embedding output get along with two planes
+        keep = any(getattr(b, "reads_history", True) for b in self.blocks)
+        planes = torch.empty((len(schedule) + 1 if keep else 2, batch.rows, self.spec.hidden), dtype=torch.float32, device=self.rt.device)
         ops.embed_gather(self.embedding, batch.ids, planes[0], scale=float(getattr(self.spec.embedding, "scale", 1.0)))
         pending = None
         for pos, entry in enumerate(schedule):
-            pending = self.blocks[entry.layer].forward(batch, planes, pos, pending, cache.view(pos))
+            kw = {"enter": self.junctions[pos]} if pos in self.junctions else {}
+            pending = self.blocks[entry.layer].forward(batch, planes, pos, pending, cache.view(pos), **kw)
         if want_rows is None or want_rows.numel() == 0:
             return None
         x = torch.empty((want_rows.numel(), self.spec.hidden), dtype=self.rt.act_dtype, device=self.rt.device)

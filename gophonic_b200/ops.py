@@ -521,7 +521,8 @@ def checked_status():
     found out of bounds since the last call (the access was skipped or redirected, nothing faulted).
     Always None in the ordinary build, whose kernels carry no checks.  Synchronises."""
     out = (c_int * 4)()
-    for name in ("rows", "cache", "attention_simt", "attention_mma", "attention_tc5", "linear_state", "delta_state", "attention_sigmoid", "hyper", "postnorm", "attention_latent", "sandwich"):
+    for name in ("rows", "cache", "attention_simt", "attention_mma", "attention_tc5", "linear_state", "delta_state", "attention_sigmoid", "hyper", "postnorm", "attention_latent", "sandwich",
+                 "short_conv", "gated_delta"):
         code = int(getattr(_lib, "gb_checked_status_" + name)(out))
         if code or out[3]:
             return name, _CHECK_NAMES.get(code, f"code {code}"), out[1], out[2], out[3]
@@ -1282,7 +1283,7 @@ def attention_sigmoid(q: torch.Tensor, out: torch.Tensor, k_plane: torch.Tensor,
 class _MoeRouteParams(Structure):
     _fields_ = [("logits", c_void_p), ("logits_stride", c_int64), ("rows", c_int), ("experts", c_int), ("top", c_int),
                 ("renorm_eps", c_float), ("dense", c_void_p), ("index", c_void_p), ("weight", c_void_p), ("score_kind", c_int), ("renorm", c_int),
-                ("correction", c_void_p), ("groups", c_int), ("keep_groups", c_int)]
+                ("correction", c_void_p), ("groups", c_int), ("keep_groups", c_int), ("group_largest", c_int)]
 
 
 class _MoeRowsParams(Structure):
@@ -1292,19 +1293,21 @@ class _MoeRowsParams(Structure):
 
 
 MOE_SCORES = {"softmax": 0, "sigmoid": 1}
+MOE_GROUP_RANKS = {"two_largest": 0, "largest": 1}
 MOE_ACTS = {"relu2": 0, "swiglu": 1, "glu_clamp": 2}     # the last two are gated: an expert's gate rows, then its up rows
 
 
 def moe_route(logits: torch.Tensor, top: int, renorm_eps: float, dense: torch.Tensor, index: torch.Tensor, weight: torch.Tensor,
               score: str = "softmax", renorm: bool = True, correction: Optional[torch.Tensor] = None, groups: int = 1,
-              keep_groups: int = 1) -> None:
+              keep_groups: int = 1, group_rank: str = "two_largest") -> None:
     """Per row of ``logits`` (float32 [rows, experts]): scores (softmax over the experts, or with ``score``
     "sigmoid" the sigmoid of each logit by itself), the ``top`` largest chosen, their weights s / (sum of the
     chosen + renorm_eps), or with ``renorm`` False the scores themselves, left in ``dense`` (float32 [rows,
     experts], zeros elsewhere) and as pairs in ``index`` (int32 [rows, top]) and ``weight`` (float32 [rows, top]).
     ``correction`` (float32 [experts]): an expert is chosen by its score plus this number, its weight comes from the score.
     ``groups`` > 1: the experts form that many equal groups of neighbours and only experts of the ``keep_groups`` groups
-    whose two largest choice scores add up to most (the lower group first of equal ones) can be chosen."""
+    whose two largest choice scores add up to most (``group_rank`` "largest": whose largest is most; the lower group first of
+    equal ones) can be chosen."""
     _need(logits, "router logits", torch.float32, 2, contiguous=False)
     rows, experts = logits.shape
     _need(dense, "expert weights", torch.float32, 2)
@@ -1317,7 +1320,8 @@ def moe_route(logits: torch.Tensor, top: int, renorm_eps: float, dense: torch.Te
         if correction.numel() != experts:
             raise KernelError(f"moe_route: {correction.numel()} corrections for {experts} experts")
     p = _MoeRouteParams(logits.data_ptr(), logits.stride(0), rows, experts, top, renorm_eps, dense.data_ptr(), index.data_ptr(), weight.data_ptr(),
-                        MOE_SCORES[score], 1 if renorm else 0, 0 if correction is None else correction.data_ptr(), int(groups), int(keep_groups))
+                        MOE_SCORES[score], 1 if renorm else 0, 0 if correction is None else correction.data_ptr(), int(groups), int(keep_groups),
+                        MOE_GROUP_RANKS[group_rank])
     _check(_lib.gb_moe_route(byref(p), _stream()))
 
 
@@ -1671,6 +1675,7 @@ class _SandwichParams(Structure):
         ("norm_w", c_void_p), ("norm_eps", c_float), ("out", c_void_p), ("row_index", c_void_p),
         ("conv_w", c_void_p), ("taps", c_int), ("state", c_void_p), ("state_slot_stride", c_int64), ("row_seq", c_void_p),
         ("seq_slot", c_void_p), ("max_slots", c_int), ("rows", c_int), ("width", c_int),
+        ("y2", c_void_p), ("pair_w", c_void_p), ("pair_w2", c_void_p), ("pair_eps", c_float),
     ]
 
 
@@ -1692,7 +1697,7 @@ def sandwich_rows(base: torch.Tensor, out: torch.Tensor, norm_weight: torch.Tens
                   y_weight: Optional[torch.Tensor] = None, y_eps: float = 0.0, result: Optional[torch.Tensor] = None,
                   planes: Optional[torch.Tensor] = None, n_planes: int = 0, average: Optional[torch.Tensor] = None,
                   x_out: Optional[torch.Tensor] = None, rows: Optional[torch.Tensor] = None, conv: Optional[torch.Tensor] = None,
-                  state: Optional[torch.Tensor] = None, batch=None) -> None:
+                  state: Optional[torch.Tensor] = None, batch=None, pair=None) -> None:
     """One pass over rows of the residual (float32 [rows, width]) between two sublayers:
 
         v = base + y / sqrt(mean(y^2) + y_eps) * y_weight          (no ``y``: v = base)      -> ``result`` if given
@@ -1702,7 +1707,11 @@ def sandwich_rows(base: torch.Tensor, out: torch.Tensor, norm_weight: torch.Tens
     With ``conv`` (float32 [taps, width]; every row is then the single token of its sequence) the normed row h is convolved
     over time on its way out, out = h + sum_j conv[j] h_(t - taps + 1 + j), the earlier rows coming from ``state``
     (float32 [slots, (taps - 1) * width], oldest first), which is moved on by this token.  With ``rows`` (int32 indices)
-    out[i] is made from row rows[i] and nothing but ``out`` is written."""
+    out[i] is made from row rows[i] and nothing but ``out`` is written.  ``pair`` = (y2, w, w2, pair_eps): a sublayer that left two
+    outputs; y stands for y / sqrt(mean(y^2) + pair_eps) * w + y2 / sqrt(mean(y2^2) + pair_eps) * w2."""
+    y2, pair_w, pair_w2, pair_eps = pair if pair is not None else (None, None, None, 0.0)
+    if pair is not None and y is None:
+        raise KernelError("sandwich_rows: a second output without a first")
     _need(base, "residual", torch.float32, 2)
     _need(out, "normed rows", dim=2)
     n, width = base.shape
@@ -1715,7 +1724,8 @@ def sandwich_rows(base: torch.Tensor, out: torch.Tensor, norm_weight: torch.Tens
     if out.shape != (out_rows, width):
         raise KernelError(f"sandwich_rows: normed rows {tuple(out.shape)}, want {(out_rows, width)}")
     for t, nm, shape in ((y, "sublayer output", (n, width)), (result, "result", (n, width)), (x_out, "averaged rows", (n, width)),
-                         (norm_weight, "norm weight", (width,)), (y_weight, "output norm weight", (width,))):
+                         (norm_weight, "norm weight", (width,)), (y_weight, "output norm weight", (width,)),
+                         (y2, "second output", (n, width)), (pair_w, "first output's weight", (width,)), (pair_w2, "second output's weight", (width,))):
         if t is not None:
             _need(t, nm, torch.float32)
             if tuple(t.shape) != shape:
@@ -1739,7 +1749,8 @@ def sandwich_rows(base: torch.Tensor, out: torch.Tensor, norm_weight: torch.Tens
                         0 if rows is None else rows.data_ptr(), 0 if conv is None else conv.data_ptr(), taps,
                         0 if taps <= 1 else state.data_ptr(), 0 if taps <= 1 else state.stride(0),
                         0 if conv is None else batch.row_seq.data_ptr(), 0 if conv is None else batch.seq_slot.data_ptr(),
-                        0 if taps <= 1 else state.shape[0], out_rows, width)
+                        0 if taps <= 1 else state.shape[0], out_rows, width, 0 if y2 is None else y2.data_ptr(),
+                        0 if y2 is None else pair_w.data_ptr(), 0 if y2 is None else pair_w2.data_ptr(), pair_eps)
     _check(_lib.gb_sandwich_rows(byref(p), _code(out.dtype), _stream()))
 
 
@@ -1763,3 +1774,130 @@ def soft_cap_(logits: torch.Tensor, cap: float) -> None:
     """In place: logits = cap * tanh(logits / cap), float32."""
     _need(logits, "logits", torch.float32)
     _check(_lib.gb_soft_cap(_ptr(logits), c_int64(logits.numel()), c_float(cap), _stream()))
+
+
+# ---- the short convolution on projected heads, and the gated delta rule ------------------------------------
+class _ShortConvParams(Structure):
+    _fields_ = [
+        ("src", c_void_p), ("row_stride", c_int64), ("conv_w", c_void_p), ("bias", c_void_p), ("taps", c_int), ("channels", c_int),
+        ("state", c_void_p), ("state_slot_stride", c_int64), ("silu", c_int), ("norm", c_int), ("eps", c_float), ("q_scale", c_float),
+        ("cos_t", c_void_p), ("sin_t", c_void_p), ("rot", c_int), ("pairs", c_int), ("table_positions", c_int), ("to_cache", c_int),
+        ("out", c_void_p), ("out_stride", c_int64), ("block_table", c_void_p), ("bt_stride", c_int), ("pages", c_int),
+        ("k_plane", c_void_p), ("v_plane", c_void_p), ("row_pos", c_void_p), ("row_seq", c_void_p), ("seq_slot", c_void_p),
+        ("seq_q_start", c_void_p), ("seq_q_len", c_void_p), ("rows", c_int), ("nseq", c_int), ("q_heads", c_int), ("k_heads", c_int),
+        ("v_heads", c_int), ("d", c_int), ("dv", c_int), ("max_slots", c_int), ("max_q_len", c_int), ("vec", c_int),
+    ]
+
+
+HEAD_NORM_NONE, HEAD_NORM_RMS, HEAD_NORM_UNIT = 0, 1, 2
+
+
+def short_conv(src: torch.Tensor, out: torch.Tensor, q_heads: int, k_heads: int, v_heads: int, d: int, dv: int, conv: Optional[torch.Tensor],
+               state: Optional[torch.Tensor], batch, bias: Optional[torch.Tensor] = None, silu: bool = False, norm: int = HEAD_NORM_NONE,
+               eps: float = 0.0, q_scale: float = 1.0, cos: Optional[torch.Tensor] = None, sin: Optional[torch.Tensor] = None,
+               rotary_dim: int = 0, pairs: bool = False, planes=None) -> None:
+    """Per row of ``src`` (q heads | k heads | v heads, rows may be wider): the ``bias`` (float32 [channels]), a causal convolution over
+    time on every channel (``conv`` float32 [taps, channels], the current token's weights last; None: none) reaching back into the
+    step's earlier rows of the same sequence and, before them, into ``state`` (float32 [slots, (taps - 1) * channels], the sequence's last
+    biased rows, oldest first, left updated), silu if asked; then per q and k head the rotation (``cos``, ``sin``, ``rotary_dim``, ``pairs``),
+    the norm behind it (``HEAD_NORM_RMS``: x / sqrt(mean x^2 + eps), ``HEAD_NORM_UNIT``: x / sqrt(sum x^2 + eps)) and, on q, a factor.
+    With ``planes`` = (block_table, k_plane, v_plane) the k and v heads go to the cache at the row's position and ``out``
+    [rows, q_heads * d] receives q in the activation dtype; without, ``out`` [rows, channels] is float32 and receives all of them."""
+    _need(src, "projected rows", dim=2, contiguous=False)
+    rows = src.shape[0]
+    channels = (q_heads + k_heads) * d + v_heads * dv
+    to_cache = planes is not None
+    _need(out, "convolved heads", src.dtype if to_cache else torch.float32, 2, contiguous=False)
+    if (src.stride(1) != 1 or src.shape[1] < channels or out.stride(1) != 1
+            or tuple(out.shape) != (rows, q_heads * d if to_cache else channels)):
+        raise KernelError(f"short_conv: rows {tuple(src.shape)}, out {tuple(out.shape)} for {q_heads} + {k_heads} heads of {d} and {v_heads} of {dv}")
+    taps = 1
+    if conv is not None:
+        taps = _conv_state(conv, state, channels, "short_conv")
+    if bias is not None:
+        _need(bias, "projection bias", torch.float32, 1)
+        if bias.numel() != channels:
+            raise KernelError(f"short_conv: a bias of {bias.numel()} for {channels} channels")
+    positions = 0
+    if rotary_dim > 0:
+        _need(cos, "rope cos", torch.float32, 2)
+        _need(sin, "rope sin", torch.float32, 2)
+        if cos.shape[1] != rotary_dim // 2 or sin.shape != cos.shape:
+            raise KernelError(f"short_conv: angle tables {tuple(cos.shape)} for rotary width {rotary_dim}")
+        positions = cos.shape[0]
+    table, k_plane, v_plane = planes if to_cache else (None, None, None)
+    if to_cache:
+        for t, nm, n, nh in ((k_plane, "key plane", d, k_heads), (v_plane, "value plane", dv, v_heads)):
+            _need(t, nm, src.dtype, 4)
+            if tuple(t.shape[1:]) != (nh, PAGE, n):
+                raise KernelError(f"short_conv: {nm} {tuple(t.shape)} for {nh} heads of {n}")
+        _need(table, "block table", torch.int32, 2)
+    has_state = taps > 1
+    p = _ShortConvParams(src.data_ptr(), src.stride(0), 0 if conv is None else conv.data_ptr(), 0 if bias is None else bias.data_ptr(), taps, channels,
+                         state.data_ptr() if has_state else 0, state.stride(0) if has_state else 0, 1 if silu else 0, int(norm), eps, q_scale,
+                         0 if rotary_dim <= 0 else cos.data_ptr(), 0 if rotary_dim <= 0 else sin.data_ptr(), int(rotary_dim), 1 if pairs else 0, positions,
+                         1 if to_cache else 0, out.data_ptr(), out.stride(0), table.data_ptr() if to_cache else 0, table.stride(0) if to_cache else 0,
+                         k_plane.shape[0] if to_cache else 0, k_plane.data_ptr() if to_cache else 0, v_plane.data_ptr() if to_cache else 0,
+                         batch.row_pos.data_ptr() if to_cache or rotary_dim > 0 else 0, batch.row_seq.data_ptr(), batch.seq_slot.data_ptr(),
+                         batch.seq_q_start.data_ptr(), batch.seq_q_len.data_ptr(), rows, batch.nseq, q_heads, k_heads, v_heads, d, dv,
+                         table.shape[0] if to_cache else (state.shape[0] if has_state else 1 << 30), int(batch.max_q_len), 0)
+    _check(_lib.gb_short_conv(byref(p), _code(src.dtype), _stream()), 2 if has_state and batch.max_q_len != 1 else 1)
+
+
+class _GatedDeltaParams(Structure):
+    _fields_ = [
+        ("rows_in", c_void_p), ("row_stride", c_int64), ("q_off", c_int), ("k_off", c_int), ("v_off", c_int),
+        ("decay_in", c_void_p), ("decay_stride", c_int64), ("dt_bias", c_void_p), ("a_log", c_void_p), ("beta_in", c_void_p), ("beta_stride", c_int64),
+        ("decay_out", c_void_p), ("coef", c_void_p), ("state", c_void_p), ("slot_stride", c_int64), ("head_stride", c_int64),
+        ("out", c_void_p), ("out_stride", c_int64), ("row_seq", c_void_p), ("seq_slot", c_void_p), ("seq_q_start", c_void_p), ("seq_q_len", c_void_p),
+        ("rows", c_int), ("nseq", c_int), ("heads", c_int), ("kv_heads", c_int), ("d", c_int), ("dv", c_int),
+        ("per_channel", c_int), ("max_slots", c_int), ("max_q_len", c_int), ("narrow_below", c_int),
+    ]
+
+
+GATED_DELTA_NARROW = 296     # fewer (head, 16 value columns) pairs than this: two columns a warp, twice the CTAs
+
+
+def gated_delta(qkv: torch.Tensor, heads: int, kv_heads: int, d: int, dv: int, decay: torch.Tensor, dt_bias: torch.Tensor, a_log: torch.Tensor,
+                beta: torch.Tensor, state: torch.Tensor, out: torch.Tensor, batch, narrow_below: Optional[int] = None) -> None:
+    """The gated delta rule over the rows of a step, in order, for every (sequence, head):
+    S <- diag(g) S, u = b (v - S^T k), S <- S + k u^T, o = S^T q.  ``qkv`` (float32, from ``short_conv``) holds kv_heads unit q heads
+    (scaled), kv_heads unit k heads, both d wide, and heads v heads of dv; head h reads q/k head h // (heads / kv_heads).
+    ``decay`` (float32 pre-activations, a free row stride): [rows, heads * d], a decay per head and key channel, or [rows, heads], one per
+    head; g = exp(-exp(a_log[h]) softplus(decay + dt_bias)).  ``beta`` (float32 [rows, heads]): b = sigmoid(beta).  ``state`` float32
+    [slots, heads, d * dv] is read and left updated, ``out`` float32 [rows, heads * dv] receives the sums."""
+    _need(qkv, "unit heads", torch.float32, 2, contiguous=False)
+    _need(state, "state", torch.float32, 3)
+    _need(out, "gated_delta out", torch.float32, 2)
+    rows = qkv.shape[0]
+    if (qkv.stride(1) != 1 or qkv.shape[1] < 2 * kv_heads * d + heads * dv or tuple(out.shape) != (rows, heads * dv) or state.shape[1] != heads
+            or state.shape[2] < d * dv or kv_heads <= 0 or heads % kv_heads):
+        raise KernelError(f"gated_delta: rows {tuple(qkv.shape)}, state {tuple(state.shape)}, out {tuple(out.shape)} for {heads} heads over "
+                          f"{kv_heads} of {d} x {dv}")
+    _need(decay, "decay pre-activations", torch.float32, 2, contiguous=False)
+    _need(beta, "write strengths", torch.float32, 2, contiguous=False)
+    _need(a_log, "decay rates", torch.float32, 1)
+    _need(dt_bias, "decay bias", torch.float32, 1)
+    per_channel = dt_bias.numel() != heads      # (with one key channel the two are the same)
+    want = heads * d if per_channel else heads
+    if (tuple(decay.shape) != (rows, want) or dt_bias.numel() != want or a_log.numel() != heads or tuple(beta.shape) != (rows, heads)
+            or decay.stride(1) != 1 or beta.stride(1) != 1):
+        raise KernelError(f"gated_delta: decays {tuple(decay.shape)} with a bias of {dt_bias.numel()}, rates of {a_log.numel()}, strengths "
+                          f"{tuple(beta.shape)} for {heads} heads of {d}")
+    single = int(batch.max_q_len) == 1
+    factors = coef = None
+    if not single:
+        factors = torch.empty((rows, want), dtype=torch.float32, device=qkv.device)
+        coef = torch.empty((rows, heads, 8), dtype=torch.float32, device=qkv.device)
+    p = _GatedDeltaParams(qkv.data_ptr(), qkv.stride(0), 0, kv_heads * d, 2 * kv_heads * d, decay.data_ptr(), decay.stride(0), dt_bias.data_ptr(),
+                          a_log.data_ptr(), beta.data_ptr(), beta.stride(0), 0 if single else factors.data_ptr(), 0 if single else coef.data_ptr(),
+                          state.data_ptr(), state.stride(0), state.stride(1), out.data_ptr(), out.stride(0), batch.row_seq.data_ptr(),
+                          batch.seq_slot.data_ptr(), batch.seq_q_start.data_ptr(), batch.seq_q_len.data_ptr(), rows, batch.nseq, heads, kv_heads, d, dv,
+                          1 if per_channel else 0, state.shape[0], int(batch.max_q_len), GATED_DELTA_NARROW if narrow_below is None else int(narrow_below))
+    _check(_lib.gb_gated_delta(byref(p), _stream()), 1 if single else 2)
+
+
+def gelu(z: torch.Tensor) -> None:
+    """In place: z times the normal law's distribution function at z (the exact gelu), computed in float32."""
+    _need(z, "gelu rows")
+    _check(_lib.gb_gelu(_ptr(z), c_int64(z.numel()), _code(z.dtype), _stream()))

@@ -10,7 +10,7 @@ A *part* is one of: mixer, feed-forward, norm, position encoding, block.  A part
 * its forward method (see each category below).
 
 A mixer additionally says what it needs from the cache, per sequence:
-``cache_request(spec) -> KVRequest | StateRequest | KVStateRequest | None`` (classmethod).
+``cache_request(spec) -> KVRequest | StateRequest | KVStateRequest | PartsRequest | None`` (classmethod).
 
 No part receives the model or its configuration: sizes and constants arrive in the part's own
 spec.
@@ -75,6 +75,13 @@ class BlockStateRequest:
     the mixer's view as ``view.mixer`` and the state as ``view.state``."""
     mixer: object
     state: StateRequest
+
+
+@dataclass(frozen=True)
+class PartsRequest:
+    """What a mixer made of several pieces, or with several states, asks for: one request a piece (any of the above, None, or
+    again such a list).  The run's view has the pieces' views as ``view.parts``, in order."""
+    parts: Tuple[object, ...]
 
 
 @dataclass
@@ -190,6 +197,10 @@ class Mixer(Part):
 
     def prepare(self, capacity: int) -> None:
         pass
+
+    def mixers(self) -> List["Part"]:
+        """The parts whose ``plan`` a step asks for: this one, or the pieces of a mixer made of several."""
+        return [self]
 
     def plan(self, nseq: int, max_q_len: int, max_kv_len: int, sm_count: int):
         """How this mixer will launch a step of ``nseq`` sequences that bring at most ``max_q_len``

@@ -1,6 +1,7 @@
 """Dense feed-forwards beside the gated SiLU one.
 
 ``ReluSquared`` (``ReluSquaredSpec``): out = down(relu(up(x))^2).
+``Gelu`` (``GeluSpec``): out = down(gelu(up(x))), the exact gelu.
 ``ClampedGLU`` (``ClampedGLUSpec``): out = down(g sigmoid(slope g) (u + 1)) with g = min(gate(x), limit) and
 u = clamp(up(x), -limit, limit); gate and up are one product, the activation is computed in float32.
 """
@@ -33,8 +34,16 @@ class ReluSquared(FeedForward):
         ops = self.rt.ops
         act = torch.empty((x.shape[0], self.spec.intermediate), dtype=x.dtype, device=x.device)
         ops.gemm(x, self.up, act)
-        ops.relu2(act)
+        self._activate(act)
         ops.gemm(act, self.down, out)
+
+    def _activate(self, act: torch.Tensor) -> None:
+        self.rt.ops.relu2(act)
+
+
+class Gelu(ReluSquared):
+    def _activate(self, act: torch.Tensor) -> None:
+        self.rt.ops.gelu(act)
 
 
 class ClampedGLU(FeedForward):

@@ -1,11 +1,14 @@
 """Grouped-query attention with a kept-first-tokens window, a softmax sink (a unit, or a learned score
 per head), biased projections, a norm of q and k (per head, or over the whole projection), an output gate
-and, optionally, another layer's keys and values (``GatedAttentionSpec``); each of them can be left off.
+a short convolution over time behind the projections, and, optionally, another layer's keys and values (``GatedAttentionSpec``); each
+of them can be left off.
 
 Per row: q | k | v | g = x [Wq; Wk; Wv; Wg]^T in one product (a layer that reads another layer's
 cache has only q and g); biases, the norm of q and k, their position encoding and the cache write in
 one row-wise kernel (a layer whose values are its keys as projected has no v: the kernel stores the key twice, before and
-behind norm and rotation); scores (q . k) * scale in float32 over the keys j <= i with i - j < window or
+behind norm and rotation; with a convolution, or a norm that stands behind a rotation which scales what it turns, that kernel is
+``ops.short_conv``, which takes the bias, the convolution with the sequence's last projected rows, the rotation and the norm in that
+order and leaves the queries in a buffer of their own); scores (q . k) * scale in float32 over the keys j <= i with i - j < window or
 j < keep_first, softmax with one more term in the denominator; the heads, each ``value_dim`` wide,
 times sigmoid(g); out = ctx Wo^T (+ bo).  Keys are cached after rotation, so a layer that shares them
 rotates only its queries.
@@ -18,7 +21,7 @@ import torch
 
 from .. import registry
 from .attention import Attention
-from .base import KVRequest, Runtime, TensorDecl
+from .base import KVRequest, KVStateRequest, Runtime, StateRequest, TensorDecl
 from .rope import scaled_magnitude
 
 
@@ -49,6 +52,8 @@ class GatedAttention(Attention):
                 decls.append(TensorDecl(prefix + n[key], (size, spec.hidden)))
                 if spec.bias:
                     decls.append(TensorDecl(prefix + n[key] + spec.bias_suffix, (size,), role="vector"))
+        if cls._taps(spec) > 0:
+            decls += [TensorDecl(prefix + n[key] + spec.conv_suffix, (size, spec.conv_taps)) for key, size in (("q", qd), ("k", kd), ("v", vd))]
         if spec.gate:
             decls.append(TensorDecl(prefix + n["g"], (od, spec.hidden)))
         if getattr(spec, "qk_norm", None) is not None and getattr(spec, "qk_norm_weight", True):
@@ -63,10 +68,19 @@ class GatedAttention(Attention):
             decls.append(TensorDecl(prefix + n["o"] + spec.bias_suffix, (spec.hidden,), role="vector"))
         return decls
 
+    @staticmethod
+    def _taps(spec) -> int:
+        return int(getattr(spec, "conv_taps", 0))
+
     @classmethod
     def cache_request(cls, spec):
         # every key is kept (the window is a mask), so layers with different windows share a group
-        return KVRequest(kv_heads=spec.kv_heads, head_dim=spec.head_dim, window=0, value_dim=spec.value_dim)
+        kv = KVRequest(kv_heads=spec.kv_heads, head_dim=spec.head_dim, window=0, value_dim=spec.value_dim)
+        taps = cls._taps(spec)
+        if taps <= 1:
+            return kv
+        channels = (spec.heads + spec.kv_heads) * spec.head_dim + spec.kv_heads * spec.value_dim
+        return KVStateRequest(kv, StateRequest(shape=((taps - 1) * channels,), dtype=torch.float32))
 
     def __init__(self, spec, prefix: str, tensors: Mapping[str, torch.Tensor], runtime: Runtime):
         if spec.heads % spec.kv_heads:
@@ -115,10 +129,20 @@ class GatedAttention(Attention):
         if getattr(spec, "out_bias", False):
             self.o_bias = tensors[prefix + n["o"] + spec.bias_suffix].to(torch.float32).contiguous()
         self.position = registry.part_class("position", spec.position.kind)(spec.position, prefix, tensors, runtime)
-        if getattr(spec, "qk_norm_after", False) and (getattr(spec, "qk_norm_weight", True)
-                                                      or scaled_magnitude(getattr(spec.position, "scaling", None)) != 1.0):
-            raise ValueError(f"{prefix}: a norm behind the position encoding is built for norms without a weight and encodings that keep "
-                             f"a head's length")
+        after = bool(getattr(spec, "qk_norm_after", False))
+        if after and getattr(spec, "qk_norm_weight", True):
+            raise ValueError(f"{prefix}: a norm behind the position encoding is built for norms without a weight")
+        # the kernel that convolves and norms behind the rotation; with neither the two orders of norm and rotation are one function
+        self.taps = self._taps(spec)
+        self.convolves = self.taps > 0 or (after and scaled_magnitude(getattr(spec.position, "scaling", None)) != 1.0)
+        if self.convolves and (not spec.own_kv or self.value_from_key or self.norm_span or (self.q_norm is not None and not after)):
+            raise ValueError(f"{prefix}: a convolution, or a norm behind a rotation that changes a head's length, is built for keys and values of the "
+                             f"layer's own and for norms head by head behind the rotation")
+        self.conv = self.all_biases = None
+        if self.taps > 0:      # [taps, channels]: a tap's weights lie together
+            self.conv = torch.cat([tensors[prefix + n[key] + spec.conv_suffix] for key in ("q", "k", "v")], dim=0).to(torch.float32).t().contiguous()
+        if self.convolves and self.biases is not None:
+            self.all_biases = torch.cat(self.biases).contiguous()
         self.q_dim = spec.heads * spec.head_dim
         self.kv_heads_own = spec.kv_heads if spec.own_kv else 0
         self.k_dim = self.kv_heads_own * spec.head_dim
@@ -160,6 +184,25 @@ class GatedAttention(Attention):
 
     def _gated_heads(self, batch, x: torch.Tensor, cache) -> torch.Tensor:
         """Everything up to the output projection: [rows, heads * value_dim] in the activation dtype."""
+        qkvg = torch.empty((x.shape[0], self.qkv.shape[0]), dtype=x.dtype, device=x.device)
+        self.rt.ops.gemm(x, self.qkv, qkvg)
+        return self.heads_of(batch, x, qkvg, cache)
+
+    # what a mixer that runs this one beside another needs: the matrix of the first product, its continuation from that product's
+    # rows, and the output projection
+    @property
+    def in_matrix(self) -> torch.Tensor:
+        return self.qkv
+
+    @in_matrix.setter
+    def in_matrix(self, w: torch.Tensor) -> None:
+        self.qkv = w
+
+    def project_out(self, heads: torch.Tensor, out: torch.Tensor) -> None:
+        self.rt.ops.gemm(heads, self.o, out, bias=self.o_bias)
+
+    def heads_of(self, batch, x: torch.Tensor, qkvg: torch.Tensor, cache) -> torch.Tensor:
+        """The (gated) heads from the projected rows ``qkvg`` (q | k | v | g, overwritten; rows may lie further apart)."""
         ops, s = self.rt.ops, self.spec
         rows = x.shape[0]
         if cache is None:
@@ -168,17 +211,22 @@ class GatedAttention(Attention):
             raise ValueError(f"attention: cache holds {cache.k.dtype}, activations are {x.dtype}")
         if cache.writable != s.own_kv:
             raise ValueError("attention: a layer with keys of its own writes its cache plane, a layer without reads another's")
-        qkvg = torch.empty((rows, self.qkv.shape[0]), dtype=x.dtype, device=x.device)
-        ops.gemm(x, self.qkv, qkvg)
         cos, sin, rot = self.position.kernel_args()
-        ops.qk_norm_rope_kv_write(qkvg, s.heads, self.kv_heads_own, s.head_dim, self.q_norm, self.k_norm, self.eps, cos, sin, rot,
-                                  batch.row_pos, batch.row_seq, batch.seq_slot, cache.block_table, cache.k if s.own_kv else None,
-                                  cache.v if s.own_kv else None, s.own_kv, biases=self.biases,
-                                  pairs=bool(getattr(self.position, "pairs", False)), value_dim=s.value_dim, span=self.norm_span,
-                                  value_from_key=self.value_from_key)
+        q = qkvg
+        if self.convolves:
+            q = torch.empty((rows, self.q_dim), dtype=x.dtype, device=x.device)
+            ops.short_conv(qkvg, q, s.heads, s.kv_heads, s.kv_heads, s.head_dim, s.value_dim, self.conv, getattr(cache, "state", None), batch,
+                           bias=self.all_biases, norm=ops.HEAD_NORM_NONE if self.q_norm is None else ops.HEAD_NORM_RMS, eps=self.eps, cos=cos, sin=sin,
+                           rotary_dim=rot, pairs=bool(getattr(self.position, "pairs", False)), planes=(cache.block_table, cache.k, cache.v))
+        else:
+            ops.qk_norm_rope_kv_write(qkvg, s.heads, self.kv_heads_own, s.head_dim, self.q_norm, self.k_norm, self.eps, cos, sin, rot,
+                                      batch.row_pos, batch.row_seq, batch.seq_slot, cache.block_table, cache.k if s.own_kv else None,
+                                      cache.v if s.own_kv else None, s.own_kv, biases=self.biases,
+                                      pairs=bool(getattr(self.position, "pairs", False)), value_dim=s.value_dim, span=self.norm_span,
+                                      value_from_key=self.value_from_key)
         ctx = torch.empty((rows, self.o_dim), dtype=x.dtype, device=x.device)
         splits, scratch = self.key_splits(batch)
-        ops.attention(qkvg, ctx, cache.k, cache.v, cache.block_table, batch.seq_slot, batch.seq_q_start, batch.seq_q_len,
+        ops.attention(q, ctx, cache.k, cache.v, cache.block_table, batch.seq_slot, batch.seq_q_start, batch.seq_q_len,
                       batch.seq_kv_len, batch.nseq, batch.max_q_len, s.heads, s.kv_heads, s.head_dim, float(s.scale), int(s.window),
                       splits, scratch, value_dim=s.value_dim, keep_first=int(s.keep_first), sink=bool(s.sink) or self.sinks is not None,
                       sinks=self.sinks)

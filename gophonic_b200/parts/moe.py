@@ -83,6 +83,7 @@ class MoE(FeedForward):
         if getattr(spec, "correction", False):
             self.correction = tensors[prefix + spec.correction_name].to(torch.float32).contiguous()
         self.groups, self.keep_groups = int(getattr(spec, "groups", 1)), int(getattr(spec, "keep_groups", 1))
+        self.group_rank = getattr(spec, "group_rank", "two_largest")
         shared = getattr(spec, "shared", None)
         self.shared = None if shared is None else registry.part_class("feed_forward", shared.kind)(shared, prefix + spec.shared_prefix, tensors, runtime)
         self.shared_gated = shared is not None and bool(getattr(spec, "shared_gate", False))
@@ -127,7 +128,7 @@ class MoE(FeedForward):
         index = torch.empty((rows, s.top), dtype=torch.int32, device=x.device)
         weight = torch.empty((rows, s.top), dtype=torch.float32, device=x.device)
         ops.moe_route(logits, s.top, float(s.renorm_eps), dense, index, weight, score=self.score, renorm=self.renorm,
-                      correction=self.correction, groups=self.groups, keep_groups=self.keep_groups)
+                      correction=self.correction, groups=self.groups, keep_groups=self.keep_groups, group_rank=self.group_rank)
         if rows <= self.ROWS_SPARSE and s.top < s.experts:
             if rows * s.top <= s.experts:      # hardly two pairs with one expert: a pair reads its expert's matrices
                 ops.moe_rows(x, self.up, self.down, index, weight, out, s.experts, s.intermediate, weight_input=self.weight_input, **kw)

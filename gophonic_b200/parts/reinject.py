@@ -1,4 +1,6 @@
-"""Junction ``reinject`` (``ReinjectSpec``): where a pass through repeated layers begins, the residual is mixed
+"""Junctions: what happens to the residual where a pass through repeated layers begins.
+
+``Reinject`` (``ReinjectSpec``): where a pass through repeated layers begins, the residual is mixed
 with the embedding output and the pass's own vector is added,
 
     x <- W [x; x0] + steps[index].
@@ -8,6 +10,10 @@ activation dtype, one product makes the new float32 residual and adds the vector
 steps, by a row-wise kernel otherwise).  The old
 residual is not needed afterwards.  A junction is built once per schedule position that names it; positions that
 name the same tensors share them.
+
+``AddStart`` (``AddStartSpec``): the embedding output is added, x <- x + x0.  For blocks that keep the results of all runs as planes
+(plane 0 is the embedding output) it only names the planes and their weights: the row-wise kernel with which the next block
+opens takes the weighted sum on its way.
 """
 from __future__ import annotations
 
@@ -47,4 +53,26 @@ class Reinject(Part):
         ops.concat_cast(h, pending if isinstance(pending, torch.Tensor) else None, x0, joined)
         out = torch.empty((rows, hidden), dtype=torch.float32, device=h.device)
         ops.gemm(joined, self.weight, out, bias=self.step)
+        return out
+
+
+class AddStart(Part):
+    category = "junction"
+    capturable = True
+
+    def __init__(self, spec, prefix: str, tensors: Mapping[str, torch.Tensor], runtime: Runtime):
+        self.spec = spec
+        self.rt = runtime
+        self.weights = torch.ones(2, dtype=torch.float32, device=runtime.device)
+
+    def over_planes(self):
+        """(number n of planes, weights [n + 1]): what goes on is sum over j < n of weights[j] planes[j] + weights[n] x."""
+        return 1, self.weights
+
+    def forward(self, batch, h: torch.Tensor, pending, x0: torch.Tensor):
+        ops = self.rt.ops
+        out = x0.clone()
+        ops.add_rows(out, h)
+        if isinstance(pending, torch.Tensor):
+            ops.add_rows(out, pending)
         return out

@@ -2,7 +2,8 @@
 over the depth behind it (``SandwichLayerSpec``).
 
 The model keeps the results of all layer runs as float32 planes [runs + 1, rows, width]: plane 0 is the embedding output
-X_0, plane i + 1 the result of the layer run at place i of the schedule.  A sublayer's output is not added when it is there but
+X_0, plane i + 1 the result of the layer run at place i of the schedule.  Where no block weighs earlier results there are two planes:
+the embedding output, and one that holds the latest result.  A sublayer's output is not added when it is there but
 handed on, with the norm that stands behind it, to the row-wise kernel that reads the residual next
 (``ops.sandwich_rows``): behind the mixer that kernel adds the normed output and norms the sum for the feed-forward;
 behind a layer the next block's (or the model's last step) adds it, stores the layer's result in its plane, forms the
@@ -10,6 +11,10 @@ weighted sum of the planes and norms it, in one pass over the row.  In a step of
 the next mixer's convolution, whose earlier inputs are then all in the sequence's state, and moves that state on; in a
 prompt the normed rows are written once in float32 and a second kernel convolves them (``ops.conv_rows``), reaching back
 into the step's own rows of the sequence and, before them, into the state.
+
+A mixer that leaves two outputs to be normed apart and added (``forward_pair``) has that done by the same kernel on its way, and a
+junction that adds planes to the residual where a pass through repeated layers begins (``over_planes``) is a weighted sum like a
+layer's own.
 
 The residual, the averages, the norms, the convolution's inputs and its state are float32; what the sublayers read is in
 the activation dtype.
@@ -34,6 +39,7 @@ class PendingResult:
     base: torch.Tensor
     at: int
     average: Optional[torch.Tensor]
+    pair: Optional[tuple] = None      # (second output, the two outputs' weights, eps) where ``y`` is the first of two
 
 
 class SandwichBlock(Part):
@@ -96,7 +102,12 @@ class SandwichBlock(Part):
         self.mixer.prepare(capacity)
 
     def mixers(self) -> List[Part]:
-        return [self.mixer]
+        return self.mixer.mixers() if hasattr(self.mixer, "mixers") else [self.mixer]
+
+    @property
+    def reads_history(self) -> bool:
+        """Whether this block reads results other than the latest (and the embedding output)."""
+        return self.average is not None
 
     def weight_bytes(self) -> int:
         return sum(p.weight_bytes() for p in (self.mixer, self.feed_forward) if p is not None and hasattr(p, "weight_bytes"))
@@ -110,22 +121,43 @@ class SandwichBlock(Part):
             raise ValueError(f"a weighted sum of {pending.average.numel()} results behind {pending.at} layer runs")
         return pending.average
 
-    def _open(self, batch, planes: torch.Tensor, pending: Optional[PendingResult], state: Optional[torch.Tensor]):
+    @staticmethod
+    def _plane(planes: torch.Tensor, at: int) -> torch.Tensor:
+        """The plane of result ``at`` (0: the embedding output); with two planes in all every result is the second."""
+        return planes[min(at, planes.shape[0] - 1)]
+
+    def _mix(self, batch, x: torch.Tensor, view):
+        """The mixer's output, or its first output and what ``pair`` needs of the second."""
+        if hasattr(self.mixer, "forward_pair"):
+            y, *pair = self.mixer.forward_pair(batch, x, view)
+            second, w, w2, eps = pair
+            return y, (second, w, w2, eps)
+        y = torch.empty((x.shape[0], x.shape[1]), dtype=torch.float32, device=x.device)
+        self.mixer.forward(batch, x, y, view)
+        return y, None
+
+    def _open(self, batch, planes: torch.Tensor, pending: Optional[PendingResult], state: Optional[torch.Tensor], enter=None):
         """Finish the layer before, form what this layer starts from and norm and convolve it for the mixer: (the residual
-        this layer starts from, the mixer's input)."""
+        this layer starts from, the mixer's input).  ``enter``: a junction that weighs planes into what this layer starts from."""
         ops = self.rt.ops
         rows, width = planes.shape[1], planes.shape[2]
         weight, eps = self.norms["mixer_norm"]
         kw, start = {}, planes[0]
+        n_planes, average = 0, None
         if pending is None:
             kw["base"] = start
         else:
-            result = planes[pending.at]
-            average = self._average_of(pending)
-            start = result if average is None else torch.empty((rows, width), dtype=torch.float32, device=planes.device)
-            kw = dict(base=pending.base, y=pending.y, y_weight=pending.norm[0], y_eps=pending.norm[1], result=result)
+            result = self._plane(planes, pending.at)
+            n_planes, average = pending.at, self._average_of(pending)
+            start = result
+            kw = dict(base=pending.base, y=pending.y, y_weight=pending.norm[0], y_eps=pending.norm[1], result=result, pair=pending.pair)
+        if enter is not None:
             if average is not None:
-                kw.update(planes=planes, n_planes=pending.at, average=average, x_out=start)
+                raise ValueError("a junction behind a layer that weighs the results so far is not built")
+            n_planes, average = enter.over_planes()
+        if average is not None:
+            start = torch.empty((rows, width), dtype=torch.float32, device=planes.device)
+            kw.update(planes=planes, n_planes=n_planes, average=average, x_out=start)
         x = torch.empty((rows, width), dtype=self.rt.act_dtype, device=planes.device)
         if self.conv is None or batch.max_q_len == 1:
             if self.conv is not None:
@@ -137,23 +169,22 @@ class SandwichBlock(Part):
             ops.conv_rows(normed, self.conv, state, x, batch)
         return start, x
 
-    def forward(self, batch, planes: torch.Tensor, at: int, pending: Optional[PendingResult], cache) -> PendingResult:
+    def forward(self, batch, planes: torch.Tensor, at: int, pending: Optional[PendingResult], cache, enter=None) -> PendingResult:
         """Runs the layer as run ``at`` of the schedule.  ``pending``: what the run before left (None: this is the first
-        run and starts from plane 0)."""
+        run and starts from plane 0).  ``enter``: the junction ahead of this run, if there is one."""
         ops = self.rt.ops
         rows, width = planes.shape[1], planes.shape[2]
         state, view = None, cache
         if self.conv is not None and self.conv.shape[0] > 1:
             state, view = cache.state, cache.mixer
-        start, x = self._open(batch, planes, pending, state)
-        y = torch.empty((rows, width), dtype=torch.float32, device=planes.device)
-        self.mixer.forward(batch, x, y, view)
+        start, x = self._open(batch, planes, pending, state, enter) if enter is not None else self._open(batch, planes, pending, state)
+        y, pair = self._mix(batch, x, view)
         if self.feed_forward is None:
-            return PendingResult(y, self.norms["mixer_out_norm"], start, at + 1, self.average)
-        result = planes[at + 1]      # holds the residual between the two sublayers until the result is complete
+            return PendingResult(y, self.norms["mixer_out_norm"], start, at + 1, self.average, pair)
+        result = self._plane(planes, at + 1)      # holds the residual between the two sublayers until the result is complete
         weight, eps = self.norms["feed_forward_norm"]
         out_weight, out_eps = self.norms["mixer_out_norm"]
-        ops.sandwich_rows(base=start, y=y, y_weight=out_weight, y_eps=out_eps, result=result, out=x, norm_weight=weight, eps=eps)
+        ops.sandwich_rows(base=start, y=y, y_weight=out_weight, y_eps=out_eps, result=result, out=x, norm_weight=weight, eps=eps, pair=pair)
         self.feed_forward.forward(batch, x, y)
         return PendingResult(y, self.norms["feed_forward_out_norm"], result, at + 1, self.average)
 
@@ -165,4 +196,4 @@ class SandwichBlock(Part):
         if average is not None:
             kw = dict(planes=planes, n_planes=pending.at, average=average)
         self.rt.ops.sandwich_rows(base=pending.base, y=pending.y, y_weight=pending.norm[0], y_eps=pending.norm[1], out=x_out,
-                                  norm_weight=weight, eps=eps, rows=rows, **kw)
+                                  norm_weight=weight, eps=eps, rows=rows, pair=pending.pair, **kw)

@@ -127,12 +127,14 @@ def _register_builtin() -> None:
     from .config.kalonex import KalonexConfig
     from .config.kimilix import KimilixConfig
     from .config.zenorax import ZenoraxConfig
+    from .config.lefalix import LefalixConfig
     register_architecture("Qwen3ForCausalLM", Qwen3Config, model_type="qwen3")
     register_architecture("Pugalix", PugalixConfig)
     register_architecture("Vepitar", VepitarConfig)
     register_architecture("Kalonex", KalonexConfig)
     register_architecture("Kimilix", KimilixConfig)
     register_architecture("Zenorax", ZenoraxConfig)
+    register_architecture("Lefalix", LefalixConfig)
 
 
 _register_builtin()
