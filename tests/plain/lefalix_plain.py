@@ -310,10 +310,14 @@ def tensor_shapes(cfg: dict, rank: int = 10, gate_rank: int = 14) -> Dict[str, t
     return out
 
 
-def random_weights(cfg: dict, seed: int, rank: int = 10, gate_rank: int = 14) -> Dict[str, np.ndarray]:
+def random_weights(cfg: dict, seed: int, rank: int = 10, gate_rank: int = 14, decided: bool = False) -> Dict[str, np.ndarray]:
     """Random weights whose values bfloat16 holds exactly: matrices of deviation 1/sqrt(inputs), norms, biases and sinks
-    that matter, decays from nearly one to a few tenths."""
+    that matter, decays from nearly one to a few tenths.  With ``decided`` all embeddings share a large part along one direction
+    and the routers read that direction above all, so that the experts' order is nearly the same for every token and far from a
+    tie: no rounding can turn a choice, which a layer with norms behind its sublayers would carry into every later row."""
     rng = np.random.default_rng(seed)
+    common = rng.standard_normal(cfg["width"])
+    common *= math.sqrt(cfg["width"]) / np.linalg.norm(common)
     w = {}
     for name, shape in tensor_shapes(cfg, rank, gate_rank).items():
         last = name.rsplit(".", 1)[-1]
@@ -330,7 +334,12 @@ def random_weights(cfg: dict, seed: int, rank: int = 10, gate_rank: int = 14) ->
         elif last == "sink":
             v = 1.0 + rng.standard_normal(shape)
         elif name == "embed":
-            v = rng.standard_normal(shape)
+            v = rng.standard_normal(shape) + (3.0 * common if decided else 0.0)
+        elif last == "router" and decided:      # whole groups one behind the other
+            count = (cfg["layers"][int(name[1:name.index(".")])]["mlp"]["router"].get("groups") or {"count": 1})["count"]
+            per = shape[0] // count
+            ranks = np.concatenate([r * per + rng.permutation(per) for r in rng.permutation(count)]) - shape[0] / 2.0
+            v = 0.05 * rng.standard_normal(shape) / math.sqrt(shape[-1]) + np.outer(0.8 * ranks, common) / shape[-1]
         elif last == "router":
             v = 2.0 * rng.standard_normal(shape) / math.sqrt(shape[-1])
         elif last in ("q", "k"):
