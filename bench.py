@@ -640,6 +640,54 @@ def probe(name, **opts):
             work, unit = float(rows) * heads * d * d, "state updates/s"
         else:
             work, unit = 2.0 * state.numel() * 4, "GB/s"
+    elif name in ("gated_delta_prompt", "gated_delta_head_prompt", "gated_delta_step_b64", "gated_delta_head_step_b64"):
+        # the gated delta rule, sizes as for delta_scan_prompt / delta_step_b64: a decay per key channel, or (head) per head
+        from types import SimpleNamespace
+        heads, d = 16, 128
+        prompt, channel = name.endswith("prompt"), "head" not in name
+        nseq, q_len = (1, 2048) if prompt else (64, 1)
+        rows = nseq * q_len
+        f32 = lambda *shape: torch.randn(*shape, device=dev, generator=g)
+        ints = lambda x: torch.tensor(x, dtype=torch.int32, device=dev)
+        unit = lambda t: t / t.norm(dim=-1, keepdim=True)
+        qkv = torch.cat([unit(f32(rows, heads, d)).view(rows, -1), unit(f32(rows, heads, d)).view(rows, -1), f32(rows, heads * d)], dim=1).contiguous()
+        wide = heads * d if channel else heads
+        decay, bias, rate, beta = f32(rows, wide), f32(wide) - 3.0, f32(heads), f32(rows, heads)
+        state = torch.zeros((nseq, heads, d * d), dtype=torch.float32, device=dev)
+        out = torch.empty((rows, heads * d), dtype=torch.float32, device=dev)
+        packed = SimpleNamespace(nseq=nseq, max_q_len=q_len, row_seq=ints([i // q_len for i in range(rows)]), seq_slot=ints(list(range(nseq))),
+                                 seq_q_start=ints([i * q_len for i in range(nseq)]), seq_q_len=ints([q_len] * nseq))
+        fn = lambda: ops.gated_delta(qkv, heads, heads, d, d, decay, bias, rate, beta, state, out, packed)
+        if prompt:
+            work, unit = float(rows) * heads * d * d, "state updates/s"
+        else:
+            work, unit = 2.0 * state.numel() * 4, "GB/s"
+    elif name in ("short_conv_prompt", "short_conv_cache_prompt"):
+        # the convolution on projected heads, 16384 rows of 2048 channels in sequences of 2048: silu and unit heads into float32 rows, or
+        # rotation and norm into the cache (the rows and heads of conv_qkv_prompt)
+        from types import SimpleNamespace
+        rows, W, taps, nseq, heads, kvh, d = 16384, 2048, 4, 8, 8, 4, 128
+        cached = "cache" in name
+        per = rows // nseq
+        f32 = lambda *shape: torch.randn(*shape, device=dev, generator=g)
+        ints = lambda x: torch.tensor(x, dtype=torch.int32, device=dev)
+        packed = SimpleNamespace(nseq=nseq, max_q_len=per, row_seq=ints([i // per for i in range(rows)]), row_pos=ints([i % per for i in range(rows)]),
+                                 seq_slot=ints(list(range(nseq))), seq_q_start=ints([i * per for i in range(nseq)]), seq_q_len=ints([per] * nseq))
+        src, conv, state = rnd(rows, W), f32(taps, W), torch.zeros((nseq, (taps - 1) * W), device=dev)
+        if cached:
+            pages = rows // 64
+            k, v = rnd(pages, kvh, 64, d), rnd(pages, kvh, 64, d)
+            table = torch.arange(pages, dtype=torch.int32, device=dev).reshape(nseq, pages // nseq)
+            out, angles, bias = torch.empty((rows, heads * d), dtype=bf, device=dev), torch.rand(per, d // 4, device=dev), f32(W)
+            cos, sin = torch.cos(angles), torch.sin(angles)
+            work = rows * W * (2 + 2)
+            fn = lambda: ops.short_conv(src, out, heads, kvh, kvh, d, d, conv, state, packed, bias=bias, norm=ops.HEAD_NORM_RMS, eps=1e-6, cos=cos, sin=sin,
+                                        rotary_dim=d // 2, pairs=True, planes=(table, k, v))
+        else:
+            out = torch.empty((rows, W), device=dev)
+            work = rows * W * (2 + 4)
+            fn = lambda: ops.short_conv(src, out, kvh, kvh, heads, d, d, conv, state, packed, silu=True, norm=ops.HEAD_NORM_UNIT, eps=1e-6, q_scale=0.1)
+        unit = "GB/s"
     elif name in ("sandwich_mid", "sandwich_open_4", "sandwich_open_8", "norm_scale_add_rows", "conv_rows_prompt", "conv_qkv_prompt"):
         # row-wise kernels over 16384 rows of 2048 (each operand is as large as L2): a sublayer's output joined and normed; the
         # same with a weighted sum over 4 or 8 planes; the postnorm block's kernel; the convolutions ahead of a mixer

@@ -18,9 +18,11 @@
 //
 // Columns of S are independent of one another, so the work is spread over (sequence, head, block of value columns).  A warp
 // owns CW columns, its 32 lanes the key channels (RC each); a thread keeps RC x CW state elements in registers across the
-// step.  The four tokens' 2 x 4 x CW partial sums a lane are added over the lanes by halving the values and the lanes, five
-// steps; the 4 x CW finished S^T (G k) are then broadcast, every lane solves the four small triangular systems itself, and
-// the outputs' remaining terms are added when a tile of eight tokens is written out, off the chain.
+// step.  The four tokens' partial sums a lane are added over the lanes by halving the values and the lanes; the 4 x CW finished
+// S^T (G k) are then broadcast and every lane solves the four small triangular systems itself.  A prompt of one sequence leaves
+// every scheduler one such warp, so nothing but this chain is on it: four further warps of the CTA fetch the tokens' rows, form
+// the products of decays and lay them out in shared memory a tile of eight tokens ahead, and add the outputs' remaining terms a
+// tile behind.
 //
 // Single tokens: reading and writing the state once, 16 bytes a thread and load, everything else of the token formed in the
 // same kernel.
@@ -41,79 +43,6 @@ __device__ __forceinline__ float decay_factor(float z, float rate) { return expf
 __device__ __forceinline__ float sigmoid_f(float x) { return 1.f / (1.f + expf(-x)); }
 
 // ------------------------------------------------------------------------------------------
-// preparation of a prompt's tokens, one warp per (row, head): the decay factors, and (A_t0, A_t1, A_t2, b, B_t0 .. B_t3), with
-// the indices counting the tokens of the row's four and zeros where the other token is not earlier (for B: not later).
-template <bool CHANNEL>
-__global__ void __launch_bounds__(128) gated_delta_prep_kernel(GatedDeltaParams p) {
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int64_t row = blockIdx.x;
-    const int h = blockIdx.y * 4 + warp;
-    if (h >= p.heads) return;
-    const int d = p.d, kh = h / (p.heads / p.kv_heads);
-    const int local = (int)(row - p.seq_q_start[p.row_seq[row]]);
-    const int n = local % C;                   // earlier tokens of the row's four
-    const float rate = expf(p.a_log[h]);
-    const float* q = p.rows_in + row * p.row_stride + p.q_off + kh * d;
-    const float* k = p.rows_in + row * p.row_stride + p.k_off + kh * d;
-    float a[C - 1], b[C];
-#pragma unroll
-    for (int s = 0; s < C; s++) {
-        if (s < C - 1) a[s] = 0.f;
-        b[s] = 0.f;
-    }
-    float g_head[C];       // one decay a head: of this row and of the earlier ones of its four, backwards
-    if (!CHANNEL) {
-#pragma unroll
-        for (int s = 0; s < C; s++)
-            g_head[s] = s <= n ? decay_factor(p.decay_in[(row - s) * p.decay_stride + h] + p.dt_bias[h], rate) : 1.f;
-        if (lane == 0) p.decay_out[row * p.heads + h] = g_head[0];
-    }
-    for (int c = lane; c < d; c += 32) {
-        const float qc = q[c], kc = k[c];
-        float between = 1.f;                   // the decays behind the other token up to this one
-#pragma unroll
-        for (int s = 0; s < C; s++) {          // s tokens back
-            if (s > n) break;
-            const float ks = s == 0 ? kc : k[c - s * p.row_stride];
-            if (s > 0) a[s - 1] = fmaf(kc, between * ks, a[s - 1]);
-            b[s] = fmaf(qc, between * ks, b[s]);
-            if (CHANNEL) {
-                if (s < C - 1 && (s < n || s == 0)) {
-                    const float g = decay_factor(p.decay_in[(row - s) * p.decay_stride + h * d + c] + p.dt_bias[h * d + c], rate);
-                    if (s == 0) p.decay_out[row * (int64_t)p.heads * d + h * d + c] = g;
-                    between *= g;
-                }
-            } else {
-                between *= g_head[s];
-            }
-        }
-    }
-#pragma unroll
-    for (int s = 0; s < C; s++) {
-        if (s < C - 1) a[s] = warp_sum(a[s]);
-        b[s] = warp_sum(b[s]);
-    }
-    if (lane == 0) {
-        float out[8];
-#pragma unroll
-        for (int e = 0; e < 8; e++) out[e] = 0.f;
-        out[3] = sigmoid_f(p.beta_in[row * p.beta_stride + h]);
-#pragma unroll
-        for (int e = 0; e < C; e++) {          // token e of the four is n - e tokens back
-#pragma unroll
-            for (int s = 0; s < C; s++) {
-                if (n - e != s) continue;
-                out[4 + e] = b[s];
-                if (s > 0 && e < C - 1) out[e] = a[s - 1];
-            }
-        }
-        float4* dst = reinterpret_cast<float4*>(p.coef + (row * p.heads + h) * 8);
-        dst[0] = make_float4(out[0], out[1], out[2], out[3]);
-        dst[1] = make_float4(out[4], out[5], out[6], out[7]);
-    }
-}
-
-// ------------------------------------------------------------------------------------------
 // N values a lane added over the lanes: N / 2 exchanged with the lane O away, and so on; lane l is left with the value of
 // number l * N / 32
 template <int N, int O>
@@ -131,6 +60,68 @@ __device__ __forceinline__ float add_over_lanes(float* a, int lane) {
             a[j] = keep + __shfl_xor_sync(0xffffffffu, give, O);
         }
         return add_over_lanes<N / 2, O / 2>(a, lane);
+    }
+}
+
+// ------------------------------------------------------------------------------------------
+// preparation of a prompt's tokens, one warp per (four tokens of a sequence, head): the decay factors, and for token t
+// (A_t0, A_t1, A_t2, b, B_t0 .. B_t3), with zeros where the other token is not earlier (for B: not later).
+template <bool CHANNEL>
+__global__ void __launch_bounds__(128) gated_delta_prep_kernel(GatedDeltaParams p) {
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int seq = blockIdx.z, h = blockIdx.y * 4 + warp, first = blockIdx.x * C;
+    const int q_len = p.seq_q_len[seq];
+    if (h >= p.heads || first >= q_len) return;
+    const int n = q_len - first < C ? q_len - first : C;       // tokens that are there
+    const int64_t row0 = p.seq_q_start[seq] + first;
+    const int d = p.d, H = p.heads, kh = h / (H / p.kv_heads);
+    const float rate = expf(p.a_log[h]);
+    float g_head[C];
+    if (!CHANNEL) {
+#pragma unroll
+        for (int t = 0; t < C; t++) {
+            g_head[t] = t < n ? decay_factor(p.decay_in[(row0 + t) * p.decay_stride + h] + p.dt_bias[h], rate) : 1.f;
+            if (lane == 0 && t < n) p.decay_out[(row0 + t) * H + h] = g_head[t];
+        }
+    }
+    // sums[t * 4 + s], s < t: A_ts; sums[16 + t * 4 + s], s <= t: B_ts; the rest stays zero and costs nothing but its exchange
+    float sums[32];
+#pragma unroll
+    for (int i = 0; i < 32; i++) sums[i] = 0.f;
+    for (int c = lane; c < d; c += 32) {
+        float q[C], k[C], g[C];
+#pragma unroll
+        for (int t = 0; t < C; t++) {
+            const int64_t row = row0 + (t < n ? t : n - 1);
+            const float* r = p.rows_in + row * p.row_stride + kh * d + c;
+            q[t] = r[p.q_off];
+            k[t] = t < n ? r[p.k_off] : 0.f;
+            if (CHANNEL) {
+                g[t] = decay_factor(p.decay_in[row * p.decay_stride + h * d + c] + p.dt_bias[h * d + c], rate);
+                if (t < n) p.decay_out[(row * H + h) * d + c] = g[t];
+            } else {
+                g[t] = g_head[t];
+            }
+        }
+#pragma unroll
+        for (int t = 0; t < C; t++) {
+            float between = 1.f;               // the decays behind s up to t
+#pragma unroll
+            for (int s = t; s >= 0; s--) {
+                const float ks = between * k[s];
+                if (s < t) sums[t * 4 + s] = fmaf(k[t], ks, sums[t * 4 + s]);
+                sums[16 + t * 4 + s] = fmaf(q[t], ks, sums[16 + t * 4 + s]);
+                between *= g[s];
+            }
+        }
+    }
+    const float total = add_over_lanes<32, 16>(sums, lane);    // lane l: sum number l
+    const int t = (lane & 15) >> 2, s = lane & 3;
+    if (t < n) {
+        float v = total;
+        int place = lane < 16 ? s : 4 + s;
+        if (lane < 16 && s == 3) v = sigmoid_f(p.beta_in[(row0 + t) * p.beta_stride + h]);
+        p.coef[((row0 + t) * H + h) * 8 + place] = v;
     }
 }
 
@@ -157,17 +148,30 @@ __device__ __forceinline__ void sts(float* p, const float* v) {
 }
 
 // RC: key channels a lane (32 RC >= d), CW: value columns a warp
+template <int RC, int CW>
+struct ScanShared {
+    static constexpr int D = 32 * RC, COLS = WARPS * CW;
+    struct __align__(16) Tile {
+        float gk[TT][D], gq[TT][D], kp[TT][D], gc[TT / C][D];
+        float v[TT][COLS];
+    } tile[2];
+    float u[2][TT][COLS], p2[2][TT][COLS];
+    float coef[4][TT][8];
+    float st[D][COLS + 1];
+};
+
 template <int RC, int CW, bool CHANNEL>
-__global__ void __launch_bounds__(THREADS) gated_delta_scan_kernel(GatedDeltaParams p) {
+__global__ void __launch_bounds__(2 * THREADS) gated_delta_scan_kernel(GatedDeltaParams p) {
     constexpr int D = 32 * RC, COLS = WARPS * CW;
     constexpr int V = RC < 4 ? RC : 4;           // neighbouring channels of a lane: lane l has l V .. l V + V - 1 of every 32 V
-    constexpr int NV = 2 * C * CW;               // sums of four tokens: S^T (G k), then S^T (G q), token by token
-    constexpr int ITEMS = (TT / C * D + THREADS - 1) / THREADS;   // (four tokens, channel) pieces a thread stages
-    __shared__ __align__(16) float gk_s[TT][D], gq_s[TT][D], kp_s[TT][D], gc_s[TT / C][D];
-    __shared__ __align__(16) float v_s[TT][COLS], u_s[TT][COLS], p2_s[TT][COLS], coef_s[TT][8];
-    __shared__ float st_s[D][COLS + 1];
+    constexpr int NV = C * CW;                   // sums of four tokens, token by token
+    constexpr int PER = 32 / NV;                 // lanes that are left with the same sum
+    constexpr int ITEMS = (TT / C * D + THREADS - 1) / THREADS;   // (four tokens, channel) pieces a staging thread makes
+    extern __shared__ __align__(16) unsigned char smem_raw[];
+    ScanShared<RC, CW>& sm = *reinterpret_cast<ScanShared<RC, CW>*>(smem_raw);
 
-    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int tid = threadIdx.x & (THREADS - 1), warp = tid >> 5, lane = tid & 31;
+    const bool stages = threadIdx.x >= THREADS;  // the second half of the CTA feeds the first
     const int d = p.d, dv = p.dv, H = p.heads;
     const int h = blockIdx.y, seq = blockIdx.z, kh = h / (H / p.kv_heads);
     const int j0 = blockIdx.x * COLS;
@@ -176,23 +180,19 @@ __global__ void __launch_bounds__(THREADS) gated_delta_scan_kernel(GatedDeltaPar
     if (!gb_check(slot, p.max_slots, GB_CHECK_SLOT)) slot = 0;
     float* S = p.state + (int64_t)slot * p.slot_stride + (int64_t)h * p.head_stride;
     auto channel = [&](int i) { return i / V * (32 * V) + lane * V + i % V; };
+    const int tiles = (q_len + TT - 1) / TT;
 
-    for (int idx = tid; idx < D * COLS; idx += THREADS) {
+    for (int idx = threadIdx.x; idx < D * COLS; idx += 2 * THREADS) {
         const int c = idx / COLS, jj = idx % COLS;
-        st_s[c][jj] = (c < d && j0 + jj < dv) ? S[(int64_t)c * dv + j0 + jj] : 0.f;
+        sm.st[c][jj] = (c < d && j0 + jj < dv) ? S[(int64_t)c * dv + j0 + jj] : 0.f;
     }
-    __syncthreads();
-    float st[RC][CW];
-#pragma unroll
-    for (int i = 0; i < RC; i++)
-#pragma unroll
-        for (int c = 0; c < CW; c++) st[i][c] = st_s[channel(i)][warp * CW + c];
 
-    // A tile's rows are fetched into registers while the tile before it is worked on: every load is unconditional (indices
-    // clamped), so they are all in flight at once; what is not there changes nothing (decay 1, key 0, strength 0).
+    // ---- staging: a tile's rows are fetched into registers a tile ahead of their place in shared memory; every load is
+    // unconditional (indices clamped); what is not there changes nothing (decay 1, key 0, strength 0)
     float rq[ITEMS][C], rk[ITEMS][C], rg[ITEMS][C], rv = 0.f, rcoef = 0.f;
-    auto fetch = [&](int t0) {
-        const int nt = q_len - t0 < TT ? q_len - t0 : TT;
+    auto fetch = [&](int tile) {
+        const int t0 = tile * TT, nt = q_len - t0 < TT ? q_len - t0 : TT;
+        const int64_t row0 = q_start + t0;
 #pragma unroll
         for (int e = 0; e < ITEMS; e++) {
             const int idx = tid + e * THREADS;
@@ -203,29 +203,27 @@ __global__ void __launch_bounds__(THREADS) gated_delta_scan_kernel(GatedDeltaPar
             for (int j = 0; j < C; j++) {
                 int t = ch * C + j;
                 t = t < nt ? t : nt - 1;
-                const int64_t row = q_start + t0 + t;
-                const float* r = p.rows_in + row * p.row_stride + kh * d + c;
+                const float* r = p.rows_in + (row0 + t) * p.row_stride + kh * d + c;
                 rq[e][j] = r[p.q_off];
                 rk[e][j] = r[p.k_off];
-                rg[e][j] = CHANNEL ? p.decay_out[(row * H + h) * d + c] : p.decay_out[row * H + h];
+                rg[e][j] = CHANNEL ? p.decay_out[((row0 + t) * H + h) * d + c] : p.decay_out[(row0 + t) * H + h];
             }
         }
         if (tid < TT * COLS) {
             int t = tid / COLS, jj = j0 + tid % COLS;
             t = t < nt ? t : nt - 1;
             jj = jj < dv ? jj : dv - 1;
-            rv = p.rows_in[(int64_t)(q_start + t0 + t) * p.row_stride + p.v_off + h * dv + jj];
+            rv = p.rows_in[(row0 + t) * p.row_stride + p.v_off + h * dv + jj];
         }
         if (tid < TT * 8) {
             int t = tid >> 3;
             t = t < nt ? t : nt - 1;
-            rcoef = p.coef[((int64_t)(q_start + t0 + t) * H + h) * 8 + (tid & 7)];
+            rcoef = p.coef[((row0 + t) * H + h) * 8 + (tid & 7)];
         }
     };
-    if (q_len > 0) fetch(0);
-    for (int t0 = 0; t0 < q_len; t0 += TT) {
-        const int nt = q_len - t0 < TT ? q_len - t0 : TT;
-        __syncthreads();   // the tile before is done with
+    auto place = [&](int tile) {
+        const int t0 = tile * TT, nt = q_len - t0 < TT ? q_len - t0 : TT;
+        auto& to = sm.tile[tile & 1];
 #pragma unroll
         for (int e = 0; e < ITEMS; e++) {
             const int idx = tid + e * THREADS;
@@ -239,117 +237,134 @@ __global__ void __launch_bounds__(THREADS) gated_delta_scan_kernel(GatedDeltaPar
                 rg[e][j] = there ? rg[e][j] : 1.f;
                 rk[e][j] = there ? rk[e][j] : 0.f;
                 up *= rg[e][j];
-                gk_s[t][c] = rk[e][j] * up;
-                gq_s[t][c] = there ? rq[e][j] * up : 0.f;
+                to.gk[t][c] = rk[e][j] * up;
+                to.gq[t][c] = there ? rq[e][j] * up : 0.f;
             }
-            gc_s[ch][c] = up;
+            to.gc[ch][c] = up;
             float down = 1.f;
 #pragma unroll
             for (int j = C - 1; j >= 0; j--) {
-                kp_s[ch * C + j][c] = rk[e][j] * down;
+                to.kp[ch * C + j][c] = rk[e][j] * down;
                 down *= rg[e][j];
             }
         }
         if (tid < TT * COLS) {
             const int t = tid / COLS, jj = tid % COLS;
-            v_s[t][jj] = (t < nt && j0 + jj < dv) ? rv : 0.f;
+            to.v[t][jj] = (t < nt && j0 + jj < dv) ? rv : 0.f;
         }
-        if (tid < TT * 8) coef_s[tid >> 3][tid & 7] = (tid >> 3) < nt ? rcoef : 0.f;
-        __syncthreads();
-        if (t0 + TT < q_len) fetch(t0 + TT);
+        if (tid < TT * 8) sm.coef[tile & 3][tid >> 3][tid & 7] = (tid >> 3) < nt ? rcoef : 0.f;
+    };
+    auto leave = [&](int tile) {
+        const int t0 = tile * TT, nt = q_len - t0 < TT ? q_len - t0 : TT;
+        for (int idx = tid; idx < nt * COLS; idx += THREADS) {
+            const int t = idx / COLS, jj = idx % COLS;
+            float o = sm.p2[tile & 1][t][jj];
 #pragma unroll
-        for (int ch = 0; ch < TT / C; ch++) {
-            float acc[NV];
+            for (int s = 0; s < C; s++) o = fmaf(sm.coef[tile & 3][t][4 + s], sm.u[tile & 1][t / C * C + s][jj], o);     // B is zero for later tokens
+            if (j0 + jj < dv) p.out[(int64_t)(q_start + t0 + t) * p.out_stride + h * dv + j0 + jj] = o;
+        }
+    };
+    if (stages && tiles > 0) {
+        fetch(0);
+        place(0);
+        if (tiles > 1) fetch(1);
+    }
+    __syncthreads();
+    float st[RC][CW];
+    if (!stages) {
 #pragma unroll
-            for (int j = 0; j < C; j++) {
-                float s1[CW], s2[CW];
+        for (int i = 0; i < RC; i++)
 #pragma unroll
-                for (int c = 0; c < CW; c++) s1[c] = s2[c] = 0.f;
+            for (int c = 0; c < CW; c++) st[i][c] = sm.st[channel(i)][warp * CW + c];
+    }
+    for (int tile = 0; tile < tiles; tile++) {
+        if (stages) {
+            if (tile + 1 < tiles) place(tile + 1);
+            if (tile + 2 < tiles) fetch(tile + 2);
+            if (tile > 0) leave(tile - 1);
+        } else {
+            const auto& in = sm.tile[tile & 1];
 #pragma unroll
-                for (int i = 0; i < RC; i += V) {
-                    float k4[V], q4[V];
-                    lds<V>(&gk_s[ch * C + j][channel(i)], k4);
-                    lds<V>(&gq_s[ch * C + j][channel(i)], q4);
-#pragma unroll
-                    for (int u = 0; u < V; u++)
-#pragma unroll
-                        for (int c = 0; c < CW; c++) {
-                            s1[c] = fmaf(k4[u], st[i + u][c], s1[c]);
-                            s2[c] = fmaf(q4[u], st[i + u][c], s2[c]);
-                        }
-                }
-#pragma unroll
-                for (int c = 0; c < CW; c++) {
-                    acc[j * CW + c] = s1[c];
-                    acc[C * CW + j * CW + c] = s2[c];
-                }
-            }
-            const float total = add_over_lanes<NV, 16>(acc, lane);
-            constexpr int PER = 32 / NV;              // lanes that hold the same sum
-            float u[C][CW];
-#pragma unroll
-            for (int j = 0; j < C; j++)
-#pragma unroll
-                for (int c = 0; c < CW; c++) u[j][c] = __shfl_sync(0xffffffffu, total, (j * CW + c) * PER);
-            if (lane >= 16 && lane % PER == 0) {
-                const int at = (lane - 16) / PER;
-                p2_s[ch * C + at / CW][warp * CW + at % CW] = total;
-            }
-#pragma unroll
-            for (int j = 0; j < C; j++) {
-                const float4 a4 = *reinterpret_cast<const float4*>(&coef_s[ch * C + j][0]);
-                const float aa[C - 1] = {a4.x, a4.y, a4.z};
-                float vj[CW];
-                lds<CW>(&v_s[ch * C + j][warp * CW], vj);
-#pragma unroll
-                for (int c = 0; c < CW; c++) {
-                    float t = vj[c] - u[j][c];
-#pragma unroll
-                    for (int s = 0; s < j; s++) t = fmaf(-aa[s], u[s][c], t);
-                    u[j][c] = a4.w * t;
-                }
-            }
-            if (lane == 0) {
-#pragma unroll
-                for (int j = 0; j < C; j++) sts<CW>(&u_s[ch * C + j][warp * CW], u[j]);
-            }
-#pragma unroll
-            for (int i = 0; i < RC; i += V) {
-                float g4[V];
-                lds<V>(&gc_s[ch][channel(i)], g4);
-#pragma unroll
-                for (int w = 0; w < V; w++)
-#pragma unroll
-                    for (int c = 0; c < CW; c++) st[i + w][c] *= g4[w];
+            for (int ch = 0; ch < TT / C; ch++) {
+                float a1[NV], a2[NV];
 #pragma unroll
                 for (int j = 0; j < C; j++) {
-                    float k4[V];
-                    lds<V>(&kp_s[ch * C + j][channel(i)], k4);
+#pragma unroll
+                    for (int c = 0; c < CW; c++) a1[j * CW + c] = a2[j * CW + c] = 0.f;
+#pragma unroll
+                    for (int i = 0; i < RC; i += V) {
+                        float k4[V], q4[V];
+                        lds<V>(&in.gk[ch * C + j][channel(i)], k4);
+                        lds<V>(&in.gq[ch * C + j][channel(i)], q4);
+#pragma unroll
+                        for (int w = 0; w < V; w++)
+#pragma unroll
+                            for (int c = 0; c < CW; c++) {
+                                a1[j * CW + c] = fmaf(k4[w], st[i + w][c], a1[j * CW + c]);
+                                a2[j * CW + c] = fmaf(q4[w], st[i + w][c], a2[j * CW + c]);
+                            }
+                    }
+                }
+                const float t1 = add_over_lanes<NV, 16>(a1, lane);
+                float u[C][CW];
+#pragma unroll
+                for (int j = 0; j < C; j++)
+#pragma unroll
+                    for (int c = 0; c < CW; c++) u[j][c] = __shfl_sync(0xffffffffu, t1, (j * CW + c) * PER);
+                const float t2 = add_over_lanes<NV, 16>(a2, lane);
+                if (lane % PER == 0) sm.p2[tile & 1][ch * C + lane / PER / CW][warp * CW + lane / PER % CW] = t2;
+#pragma unroll
+                for (int j = 0; j < C; j++) {
+                    const float4 a4 = *reinterpret_cast<const float4*>(&sm.coef[tile & 3][ch * C + j][0]);
+                    const float aa[C - 1] = {a4.x, a4.y, a4.z};
+                    float vj[CW];
+                    lds<CW>(&in.v[ch * C + j][warp * CW], vj);
+#pragma unroll
+                    for (int c = 0; c < CW; c++) {
+                        float t = vj[c] - u[j][c];
+#pragma unroll
+                        for (int s = 0; s < j; s++) t = fmaf(-aa[s], u[s][c], t);
+                        u[j][c] = a4.w * t;
+                    }
+                }
+#pragma unroll
+                for (int i = 0; i < RC; i += V) {
+                    float g4[V];
+                    lds<V>(&in.gc[ch][channel(i)], g4);
 #pragma unroll
                     for (int w = 0; w < V; w++)
 #pragma unroll
-                        for (int c = 0; c < CW; c++) st[i + w][c] = fmaf(k4[w], u[j][c], st[i + w][c]);
+                        for (int c = 0; c < CW; c++) st[i + w][c] *= g4[w];
+#pragma unroll
+                    for (int j = 0; j < C; j++) {
+                        float k4[V];
+                        lds<V>(&in.kp[ch * C + j][channel(i)], k4);
+#pragma unroll
+                        for (int w = 0; w < V; w++)
+#pragma unroll
+                            for (int c = 0; c < CW; c++) st[i + w][c] = fmaf(k4[w], u[j][c], st[i + w][c]);
+                    }
+                }
+                if (lane == 0) {
+#pragma unroll
+                    for (int j = 0; j < C; j++) sts<CW>(&sm.u[tile & 1][ch * C + j][warp * CW], u[j]);
                 }
             }
         }
         __syncthreads();
-        for (int idx = tid; idx < nt * COLS; idx += THREADS) {
-            const int t = idx / COLS, jj = idx % COLS;
-            float o = p2_s[t][jj];
+    }
+    if (stages) {
+        if (tiles > 0) leave(tiles - 1);
+    } else {
 #pragma unroll
-            for (int s = 0; s < C; s++) o = fmaf(coef_s[t][4 + s], u_s[t / C * C + s][jj], o);     // B is zero for later tokens
-            if (j0 + jj < dv) p.out[(int64_t)(q_start + t0 + t) * p.out_stride + h * dv + j0 + jj] = o;
-        }
+        for (int i = 0; i < RC; i++)
+#pragma unroll
+            for (int c = 0; c < CW; c++) sm.st[channel(i)][warp * CW + c] = st[i][c];
     }
     __syncthreads();
-#pragma unroll
-    for (int i = 0; i < RC; i++)
-#pragma unroll
-        for (int c = 0; c < CW; c++) st_s[channel(i)][warp * CW + c] = st[i][c];
-    __syncthreads();
-    for (int idx = tid; idx < D * COLS; idx += THREADS) {
+    for (int idx = threadIdx.x; idx < D * COLS; idx += 2 * THREADS) {
         const int c = idx / COLS, jj = idx % COLS;
-        if (c < d && j0 + jj < dv) S[(int64_t)c * dv + j0 + jj] = st_s[c][jj];
+        if (c < d && j0 + jj < dv) S[(int64_t)c * dv + j0 + jj] = sm.st[c][jj];
     }
 }
 
@@ -473,7 +488,14 @@ int launch_step(const GatedDeltaParams& p, cudaStream_t stream) {
 
 template <int RC, int CW, bool CHANNEL>
 int launch_scan(const GatedDeltaParams& p, cudaStream_t stream) {
-    gated_delta_scan_kernel<RC, CW, CHANNEL><<<dim3(ceil_div(p.dv, WARPS * CW), p.heads, p.nseq), THREADS, 0, stream>>>(p);
+    constexpr int smem = (int)sizeof(ScanShared<RC, CW>);
+    static bool configured = false;
+    if (!configured && smem > 48 * 1024) {
+        cudaError_t e = cudaFuncSetAttribute(gated_delta_scan_kernel<RC, CW, CHANNEL>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+        if (e != cudaSuccess) GB_REFUSE("gated_delta: cannot reserve %d bytes of shared memory: %s", smem, cudaGetErrorString(e));
+        configured = true;
+    }
+    gated_delta_scan_kernel<RC, CW, CHANNEL><<<dim3(ceil_div(p.dv, WARPS * CW), p.heads, p.nseq), 2 * THREADS, smem, stream>>>(p);
     GB_CHECK_LAUNCH("gated_delta_scan");
     return 0;
 }
@@ -485,8 +507,8 @@ int launch(const GatedDeltaParams& p, cudaStream_t stream) {
         const bool vec = !(p.dv & 3) && !(p.head_stride & 3) && !(p.slot_stride & 3) && !((uintptr_t)p.state & 15);
         return vec ? launch_step<4, CHANNEL>(p, stream) : launch_step<1, CHANNEL>(p, stream);
     }
-    if (!p.coef || !p.decay_out || !p.row_seq) GB_REFUSE("gated_delta: no room for the tokens' factors");
-    gated_delta_prep_kernel<CHANNEL><<<dim3(p.rows, ceil_div(p.heads, 4)), 128, 0, stream>>>(p);
+    if (!p.coef || !p.decay_out) GB_REFUSE("gated_delta: no room for the tokens' factors");
+    gated_delta_prep_kernel<CHANNEL><<<dim3(ceil_div(p.max_q_len, C), ceil_div(p.heads, 4), p.nseq), 128, 0, stream>>>(p);
     GB_CHECK_LAUNCH("gated_delta_prep");
     // few (head, column block) pairs: two columns a warp leave more CTAs, and warps, to hide one another's chains
     const bool narrow = (int64_t)p.heads * p.nseq * ceil_div(p.dv, 16) < p.narrow_below;

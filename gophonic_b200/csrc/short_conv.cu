@@ -27,7 +27,7 @@ constexpr int MAX_TAPS = 16;
 constexpr int MAX_HEAD = 256;
 constexpr int WARPS = 4;
 
-__device__ __forceinline__ float silu_f(float x) { return x / (1.f + expf(-x)); }
+__device__ __forceinline__ float silu_f(float x) { return __fdividef(x, 1.f + expf(-x)); }     // a quotient good to two units in the last place
 
 struct Pair {
     float a, b;
@@ -83,21 +83,22 @@ __device__ __forceinline__ Head head_of(const ShortConvParams& p, int hh) {
     return {2, (p.q_heads + p.k_heads) * p.d + v * p.dv, p.dv, v};
 }
 
-// activation, rotation, norm and store of one row of one head, two channels a lane and piece
-template <typename T, int NE>
-__device__ __forceinline__ void finish_head(const ShortConvParams& p, const Head& hd, int64_t row, int slot, Pair (&y)[NE], float* sh, int lane, bool vec) {
+// activation, rotation, norm and store of one row of one head, two channels a lane and piece.  CACHE: q into the buffer, k and v
+// into the cache (`bt`: the sequence's block-table row); else float32 rows.  HALF: channels i and i + rot / 2 may turn together
+template <typename T, int NE, bool CACHE, bool HALF>
+__device__ __forceinline__ void finish_head(const ShortConvParams& p, const Head& hd, int64_t row, int pos, const int* bt, Pair (&y)[NE], float* sh, int lane,
+                                            bool vec) {
     if (p.silu) {
 #pragma unroll
         for (int e = 0; e < NE; e++) y[e] = {silu_f(y[e].a), silu_f(y[e].b)};
     }
-    const int pos = p.rot > 0 || p.to_cache ? p.row_pos[row] : 0;
     if (hd.kind != 2) {
         if (p.rot > 0) {
             const int half = p.rot / 2;
             const int tpos = gb_check(pos, p.table_positions, GB_CHECK_ROPE_POSITION) ? pos : 0;
             const float* ct = p.cos_t + (int64_t)tpos * half;
             const float* st = p.sin_t + (int64_t)tpos * half;
-            if (p.pairs) {
+            if (!HALF || p.pairs) {
 #pragma unroll
                 for (int e = 0; e < NE; e++) {
                     const int j = lane + 32 * e;       // channels 2j and 2j + 1
@@ -106,7 +107,7 @@ __device__ __forceinline__ void finish_head(const ShortConvParams& p, const Head
                         y[e] = {y[e].a * c - y[e].b * s, y[e].b * c + y[e].a * s};
                     }
                 }
-            } else {
+            } else if constexpr (HALF) {
                 __syncwarp();
 #pragma unroll
                 for (int e = 0; e < NE; e++) {
@@ -132,21 +133,19 @@ __device__ __forceinline__ void finish_head(const ShortConvParams& p, const Head
 #pragma unroll
             for (int e = 0; e < NE; e++) ss = fmaf(y[e].a, y[e].a, fmaf(y[e].b, y[e].b, ss));
             ss = warp_sum(ss);
-            const float inv = 1.0f / sqrtf((p.norm == 1 ? ss / (float)hd.n : ss) + p.eps);
+            float inv = 1.0f / sqrtf((p.norm == 1 ? ss / (float)hd.n : ss) + p.eps);
+            if (hd.kind == 0) inv *= p.q_scale;
 #pragma unroll
             for (int e = 0; e < NE; e++) y[e] = {y[e].a * inv, y[e].b * inv};
-        }
-        if (hd.kind == 0 && p.q_scale != 1.f) {
+        } else if (hd.kind == 0 && p.q_scale != 1.f) {
 #pragma unroll
             for (int e = 0; e < NE; e++) y[e] = {y[e].a * p.q_scale, y[e].b * p.q_scale};
         }
     }
-    if (p.to_cache) {
-        T* dst;
-        if (hd.kind == 0) {
-            dst = (T*)p.out + row * p.out_stride + hd.c0;
-        } else {
-            const int64_t page = page_of(block_table_row(p.block_table, p.bt_stride, slot, p.max_slots), pos, p.bt_stride, p.pages);
+    if constexpr (CACHE) {
+        T* dst = (T*)p.out + row * p.out_stride + hd.c0;
+        if (hd.kind != 0) {
+            const int64_t page = page_of(bt, pos, p.bt_stride, p.pages);
             const int heads = hd.kind == 1 ? p.k_heads : p.v_heads;
             dst = (T*)(hd.kind == 1 ? p.k_plane : p.v_plane) + ((page * heads + hd.at) * GB_PAGE + (pos % GB_PAGE)) * (int64_t)hd.n;
         }
@@ -165,87 +164,12 @@ __device__ __forceinline__ void finish_head(const ShortConvParams& p, const Head
     }
 }
 
-// prompts of few taps: a warp's ROWS rows through a window of registers
-template <typename T, int ROWS, int TAPS, int NE>
-__global__ void __launch_bounds__(32 * WARPS) short_conv_window_kernel(ShortConvParams p) {
-    pdl_wait();
-    pdl_trigger();
-    __shared__ float sh[WARPS][MAX_HEAD];
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int hh = blockIdx.y * WARPS + warp;
-    if (hh >= p.q_heads + p.k_heads + p.v_heads) return;
-    const Head hd = head_of(p, hh);
-    const int64_t r0 = (int64_t)blockIdx.x * ROWS;
-    const bool vec = p.vec;
-    const T* base = (const T*)p.src + hd.c0;
-    Pair x[ROWS + TAPS - 1][NE];
-#pragma unroll
-    for (int i = 0; i < ROWS + TAPS - 1; i++) {
-        int64_t r = r0 + i - (TAPS - 1);
-        r = r < 0 ? 0 : (r < p.rows ? r : p.rows - 1);      // rows outside are replaced or not used
-#pragma unroll
-        for (int e = 0; e < NE; e++) {
-            const int c = 2 * (lane + 32 * e);
-            x[i][e] = load_pair<T>(base + r * p.row_stride + c, min(2, hd.n - c), vec);
-        }
-    }
-    Pair w[TAPS][NE], bias[NE];
-#pragma unroll
-    for (int e = 0; e < NE; e++) {
-        const int c = 2 * (lane + 32 * e), m = min(2, hd.n - c);
-        bias[e] = {0.f, 0.f};
-        if (p.bias) bias[e] = load_pair<float>(p.bias + hd.c0 + c, m, false);
-#pragma unroll
-        for (int j = 0; j < TAPS; j++) {
-            w[j][e] = {1.f, 1.f};
-            if (p.conv_w) w[j][e] = load_pair<float>(p.conv_w + (int64_t)j * p.channels + hd.c0 + c, m, false);
-        }
-    }
-#pragma unroll
-    for (int i = 0; i < ROWS; i++) {
-        const int64_t row = r0 + i;
-        if (row >= p.rows) break;
-        const int seq = p.row_seq[row];
-        const int local = (int)(row - p.seq_q_start[seq]);     // the row's place in its sequence's portion
-        int slot = p.seq_slot[seq];
-        if (!gb_check(slot, p.max_slots, GB_CHECK_SLOT)) slot = 0;
-        const float* st = p.state + (int64_t)slot * p.state_slot_stride + hd.c0;
-        Pair y[NE];
-#pragma unroll
-        for (int e = 0; e < NE; e++) {
-            const int c = 2 * (lane + 32 * e), m = min(2, hd.n - c);
-            y[e] = {0.f, 0.f};
-#pragma unroll
-            for (int j = 0; j < TAPS; j++) {
-                const int back = TAPS - 1 - j;
-                Pair u = {x[i + j][e].a + bias[e].a, x[i + j][e].b + bias[e].b};
-                if (back > local) u = load_pair<float>(st + (int64_t)(TAPS - 1 + local - back) * p.channels + c, m, false);
-                y[e] = {fmaf(w[j][e].a, u.a, y[e].a), fmaf(w[j][e].b, u.b, y[e].b)};
-            }
-        }
-        finish_head<T, NE>(p, hd, row, slot, y, sh[warp], lane, vec);
-    }
-}
-
-// one row a warp, any number of taps; for single tokens it also moves the state on
+// one row of one head with any number of taps: what the portion does not hold comes from the state
 template <typename T, int NE>
-__global__ void __launch_bounds__(32 * WARPS) short_conv_row_kernel(ShortConvParams p) {
-    pdl_wait();
-    pdl_trigger();
-    __shared__ float sh[WARPS][MAX_HEAD];
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int hh = blockIdx.y * WARPS + warp;
-    if (hh >= p.q_heads + p.k_heads + p.v_heads) return;
-    const Head hd = head_of(p, hh);
-    const int64_t row = blockIdx.x;
-    const int seq = p.row_seq[row];
-    const int local = (int)(row - p.seq_q_start[seq]);
-    int slot = p.seq_slot[seq];
-    if (!gb_check(slot, p.max_slots, GB_CHECK_SLOT)) slot = 0;
-    const bool vec = p.vec, move = p.taps > 1 && p.max_q_len == 1;
+__device__ __forceinline__ void convolve_row(const ShortConvParams& p, const Head& hd, int64_t row, int local, int slot, Pair (&y)[NE], int lane, bool vec) {
+    const bool move = p.taps > 1 && p.max_q_len == 1;
     const T* base = (const T*)p.src + hd.c0;
     float* st = p.state ? p.state + (int64_t)slot * p.state_slot_stride + hd.c0 : nullptr;
-    Pair y[NE];
 #pragma unroll
     for (int e = 0; e < NE; e++) {
         const int c = 2 * (lane + 32 * e), m = min(2, hd.n - c);
@@ -273,7 +197,97 @@ __global__ void __launch_bounds__(32 * WARPS) short_conv_row_kernel(ShortConvPar
         if (p.conv_w) w = load_pair<float>(p.conv_w + (int64_t)(p.taps - 1) * p.channels + hd.c0 + c, m, false);
         y[e] = {fmaf(w.a, own.a, y[e].a), fmaf(w.b, own.b, y[e].b)};
     }
-    finish_head<T, NE>(p, hd, row, slot, y, sh[warp], lane, vec);
+}
+
+// Prompts of few taps: a warp's ROWS rows through a window of registers.  Rows whose taps all lie in their own portion, nearly
+// all of them, take straight code; a warp that holds a portion's first rows goes row by row.
+template <typename T, int ROWS, int TAPS, int NE, bool CACHE>
+__global__ void __launch_bounds__(32 * WARPS) short_conv_window_kernel(ShortConvParams p) {
+    pdl_wait();
+    pdl_trigger();
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int hh = blockIdx.y * WARPS + warp;
+    if (hh >= p.q_heads + p.k_heads + p.v_heads) return;
+    const Head hd = head_of(p, hh);
+    const int64_t r0 = (int64_t)blockIdx.x * ROWS;
+    const int n = p.rows - r0 < ROWS ? (int)(p.rows - r0) : ROWS;
+    const bool vec = p.vec;
+    const T* base = (const T*)p.src + hd.c0;
+    Pair x[ROWS + TAPS - 1][NE];
+#pragma unroll
+    for (int i = 0; i < ROWS + TAPS - 1; i++) {
+        int64_t r = r0 + i - (TAPS - 1);
+        r = r < 0 ? 0 : (r < p.rows ? r : p.rows - 1);      // rows outside are not used
+#pragma unroll
+        for (int e = 0; e < NE; e++) {
+            const int c = 2 * (lane + 32 * e);
+            x[i][e] = load_pair<T>(base + r * p.row_stride + c, min(2, hd.n - c), vec);
+        }
+    }
+    const int seq0 = p.row_seq[r0];
+    const bool plain = p.row_seq[r0 + n - 1] == seq0 && r0 - p.seq_q_start[seq0] >= TAPS - 1;
+    if (!plain) {
+        for (int i = 0; i < n; i++) {
+            const int64_t row = r0 + i;
+            const int seq = p.row_seq[row];
+            int slot = p.seq_slot[seq];
+            if (!gb_check(slot, p.max_slots, GB_CHECK_SLOT)) slot = 0;
+            Pair y[NE];
+            convolve_row<T, NE>(p, hd, row, (int)(row - p.seq_q_start[seq]), slot, y, lane, vec);
+            finish_head<T, NE, CACHE, false>(p, hd, row, CACHE || p.rot > 0 ? p.row_pos[row] : 0,
+                                             CACHE ? block_table_row(p.block_table, p.bt_stride, slot, p.max_slots) : nullptr, y, nullptr, lane, vec);
+        }
+        return;
+    }
+    Pair w[TAPS][NE];
+#pragma unroll
+    for (int e = 0; e < NE; e++) {
+        const int c = 2 * (lane + 32 * e), m = min(2, hd.n - c);
+#pragma unroll
+        for (int j = 0; j < TAPS; j++) {
+            w[j][e] = {1.f, 1.f};
+            if (p.conv_w) w[j][e] = load_pair<float>(p.conv_w + (int64_t)j * p.channels + hd.c0 + c, m, vec);
+        }
+        if (p.bias) {
+            const Pair bias = load_pair<float>(p.bias + hd.c0 + c, m, vec);
+#pragma unroll
+            for (int i = 0; i < ROWS + TAPS - 1; i++) x[i][e] = {x[i][e].a + bias.a, x[i][e].b + bias.b};
+        }
+    }
+    const int pos0 = CACHE || p.rot > 0 ? p.row_pos[r0] : 0;      // rows of a sequence are consecutive positions
+    const int* bt = CACHE ? block_table_row(p.block_table, p.bt_stride, p.seq_slot[seq0], p.max_slots) : nullptr;
+#pragma unroll
+    for (int i = 0; i < ROWS; i++) {
+        if (i >= n) break;
+        Pair y[NE];
+#pragma unroll
+        for (int e = 0; e < NE; e++) {
+            y[e] = {0.f, 0.f};
+#pragma unroll
+            for (int j = 0; j < TAPS; j++) y[e] = {fmaf(w[j][e].a, x[i + j][e].a, y[e].a), fmaf(w[j][e].b, x[i + j][e].b, y[e].b)};
+        }
+        finish_head<T, NE, CACHE, false>(p, hd, r0 + i, pos0 + i, bt, y, nullptr, lane, vec);
+    }
+}
+
+// one row a warp, any number of taps; for single tokens it also moves the state on
+template <typename T, int NE, bool CACHE>
+__global__ void __launch_bounds__(32 * WARPS) short_conv_row_kernel(ShortConvParams p) {
+    pdl_wait();
+    pdl_trigger();
+    __shared__ float sh[WARPS][MAX_HEAD];
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int hh = blockIdx.y * WARPS + warp;
+    if (hh >= p.q_heads + p.k_heads + p.v_heads) return;
+    const Head hd = head_of(p, hh);
+    const int64_t row = blockIdx.x;
+    const int seq = p.row_seq[row];
+    int slot = p.seq_slot[seq];
+    if (!gb_check(slot, p.max_slots, GB_CHECK_SLOT)) slot = 0;
+    Pair y[NE];
+    convolve_row<T, NE>(p, hd, row, (int)(row - p.seq_q_start[seq]), slot, y, lane, p.vec);
+    finish_head<T, NE, CACHE, true>(p, hd, row, CACHE || p.rot > 0 ? p.row_pos[row] : 0,
+                                    CACHE ? block_table_row(p.block_table, p.bt_stride, slot, p.max_slots) : nullptr, y, sh[warp], lane, p.vec);
 }
 
 // the last taps - 1 rows u of every sequence's portion into its state; a portion shorter than that pushes the older rows on
@@ -299,21 +313,21 @@ __global__ void short_conv_state_kernel(ShortConvParams p) {
 constexpr int WINDOW_ROWS = 8;
 constexpr int WINDOW_MIN_ROWS = 96;    // packed rows from which a warp takes eight of them
 
-template <typename T, int NE>
+template <typename T, int NE, bool CACHE>
 int launch_ne(const ShortConvParams& p, cudaStream_t stream) {
     const int heads = p.q_heads + p.k_heads + p.v_heads;
     const int hy = ceil_div(heads, WARPS);
     if (hy > 65535) GB_REFUSE("short_conv: %d heads exceed one launch", heads);
-    if (p.max_q_len != 1 && p.taps <= 4 && p.rows >= WINDOW_MIN_ROWS) {
+    if (p.max_q_len != 1 && p.taps <= 4 && p.rows >= WINDOW_MIN_ROWS && (p.rot == 0 || p.pairs)) {
         const dim3 grid(ceil_div(p.rows, WINDOW_ROWS), hy), block(32 * WARPS);
         switch (p.taps) {
-            case 1: launch_pdl(short_conv_window_kernel<T, WINDOW_ROWS, 1, NE>, grid, block, 0, stream, p); break;
-            case 2: launch_pdl(short_conv_window_kernel<T, WINDOW_ROWS, 2, NE>, grid, block, 0, stream, p); break;
-            case 3: launch_pdl(short_conv_window_kernel<T, WINDOW_ROWS, 3, NE>, grid, block, 0, stream, p); break;
-            default: launch_pdl(short_conv_window_kernel<T, WINDOW_ROWS, 4, NE>, grid, block, 0, stream, p); break;
+            case 1: launch_pdl(short_conv_window_kernel<T, WINDOW_ROWS, 1, NE, CACHE>, grid, block, 0, stream, p); break;
+            case 2: launch_pdl(short_conv_window_kernel<T, WINDOW_ROWS, 2, NE, CACHE>, grid, block, 0, stream, p); break;
+            case 3: launch_pdl(short_conv_window_kernel<T, WINDOW_ROWS, 3, NE, CACHE>, grid, block, 0, stream, p); break;
+            default: launch_pdl(short_conv_window_kernel<T, WINDOW_ROWS, 4, NE, CACHE>, grid, block, 0, stream, p); break;
         }
     } else {
-        launch_pdl(short_conv_row_kernel<T, NE>, dim3(p.rows, hy), dim3(32 * WARPS), 0, stream, p);
+        launch_pdl(short_conv_row_kernel<T, NE, CACHE>, dim3(p.rows, hy), dim3(32 * WARPS), 0, stream, p);
     }
     GB_CHECK_LAUNCH("short_conv");
     if (p.taps > 1 && p.max_q_len != 1) {
@@ -328,10 +342,11 @@ int launch(ShortConvParams p, cudaStream_t stream) {
     const uintptr_t pair = 2 * sizeof(T) - 1;
     p.vec = !(p.d & 1) && !(p.dv & 1) && !(p.row_stride & 1) && !((uintptr_t)p.src & pair) && !(p.out_stride & 1) &&
             !((uintptr_t)p.out & (p.to_cache ? pair : 7)) && !(((uintptr_t)p.k_plane | (uintptr_t)p.v_plane) & pair);
+    p.vec = p.vec && !(((uintptr_t)p.conv_w | (uintptr_t)p.bias) & 7);
     const int most = p.d > p.dv ? p.d : p.dv;
-    if (most <= 64) return launch_ne<T, 1>(p, stream);
-    if (most <= 128) return launch_ne<T, 2>(p, stream);
-    return launch_ne<T, 4>(p, stream);
+    if (most <= 64) return p.to_cache ? launch_ne<T, 1, true>(p, stream) : launch_ne<T, 1, false>(p, stream);
+    if (most <= 128) return p.to_cache ? launch_ne<T, 2, true>(p, stream) : launch_ne<T, 2, false>(p, stream);
+    return p.to_cache ? launch_ne<T, 4, true>(p, stream) : launch_ne<T, 4, false>(p, stream);
 }
 
 }  // namespace
