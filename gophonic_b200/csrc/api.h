@@ -454,7 +454,7 @@ struct GatedDeltaParams {
     const int* seq_q_len;
     int rows, nseq, heads, kv_heads, d, dv;
     int per_channel, max_slots, max_q_len;
-    int narrow_below;       // with fewer (head, 16 columns) pairs than this a warp takes two columns instead of four
+    int narrow_below;       // heads of up to 64 key channels: with fewer (head, 16 columns) pairs than this a warp takes two columns instead of four
 };
 GB_API int gb_gated_delta(const GatedDeltaParams* p, cudaStream_t stream);
 GB_API int gb_gelu(void* z, int64_t n, int dtype, cudaStream_t stream);

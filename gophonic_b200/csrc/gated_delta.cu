@@ -19,7 +19,7 @@
 // Columns of S are independent of one another, so the work is spread over (sequence, head, block of value columns).  A warp
 // owns CW columns, its 32 lanes the key channels (RC each); a thread keeps RC x CW state elements in registers across the
 // step.  The four tokens' partial sums a lane are added over the lanes by halving the values and the lanes; the 4 x CW finished
-// S^T (G k) are then broadcast and every lane solves the four small triangular systems itself.  A prompt of one sequence leaves
+// v - S^T (G k) are then broadcast and every lane solves the four small triangular systems itself.  A prompt of one sequence leaves
 // every scheduler one such warp, so nothing but this chain is on it: four further warps of the CTA fetch the tokens' rows, form
 // the products of decays and lay them out in shared memory a tile of eight tokens ahead, and add the outputs' remaining terms a
 // tile behind.
@@ -125,6 +125,22 @@ __global__ void __launch_bounds__(128) gated_delta_prep_kernel(GatedDeltaParams 
     }
 }
 
+// The same for lanes that hold their values in an order of their own: the values of numbers N / 2 .. N - 1 are the ones the lane O
+// away keeps, so nothing is chosen.
+template <int N, int O>
+__device__ __forceinline__ float fold_lanes(float* a) {
+    if constexpr (O == 0) {
+        return a[0];
+    } else if constexpr (N == 1) {
+        a[0] += __shfl_xor_sync(0xffffffffu, a[0], O);
+        return fold_lanes<1, O / 2>(a);
+    } else {
+#pragma unroll
+        for (int j = 0; j < N / 2; j++) a[j] += __shfl_xor_sync(0xffffffffu, a[j + N / 2], O);
+        return fold_lanes<N / 2, O / 2>(a);
+    }
+}
+
 template <int V>
 __device__ __forceinline__ void lds(const float* p, float* v) {
     if constexpr (V == 4) {
@@ -180,6 +196,9 @@ __global__ void __launch_bounds__(2 * THREADS) gated_delta_scan_kernel(GatedDelt
     if (!gb_check(slot, p.max_slots, GB_CHECK_SLOT)) slot = 0;
     float* S = p.state + (int64_t)slot * p.slot_stride + (int64_t)h * p.head_stride;
     auto channel = [&](int i) { return i / V * (32 * V) + lane * V + i % V; };
+    // A thread's slot j of the four tokens' sums is token j ^ mine_t and its column slot c is column c ^ mine_c of the warp's, so that
+    // adding over the lanes (fold_lanes) leaves each lane the sum of token mine_t and column mine_c: lane 8 j + PER c has (j, c)
+    const int mine_t = lane >> 3, mine_c = (lane / PER) % CW;
     const int tiles = (q_len + TT - 1) / TT;
 
     for (int idx = threadIdx.x; idx < D * COLS; idx += 2 * THREADS) {
@@ -190,9 +209,10 @@ __global__ void __launch_bounds__(2 * THREADS) gated_delta_scan_kernel(GatedDelt
     // ---- staging: a tile's rows are fetched into registers a tile ahead of their place in shared memory; every load is
     // unconditional (indices clamped); what is not there changes nothing (decay 1, key 0, strength 0)
     float rq[ITEMS][C], rk[ITEMS][C], rg[ITEMS][C], rv = 0.f, rcoef = 0.f;
+    const int stride = (int)p.row_stride;
     auto fetch = [&](int tile) {
         const int t0 = tile * TT, nt = q_len - t0 < TT ? q_len - t0 : TT;
-        const int64_t row0 = q_start + t0;
+        const int row0 = q_start + t0;           // products of two 32-bit numbers, one instruction an address
 #pragma unroll
         for (int e = 0; e < ITEMS; e++) {
             const int idx = tid + e * THREADS;
@@ -203,22 +223,22 @@ __global__ void __launch_bounds__(2 * THREADS) gated_delta_scan_kernel(GatedDelt
             for (int j = 0; j < C; j++) {
                 int t = ch * C + j;
                 t = t < nt ? t : nt - 1;
-                const float* r = p.rows_in + (row0 + t) * p.row_stride + kh * d + c;
+                const float* r = p.rows_in + (int64_t)(row0 + t) * stride + kh * d + c;
                 rq[e][j] = r[p.q_off];
                 rk[e][j] = r[p.k_off];
-                rg[e][j] = CHANNEL ? p.decay_out[((row0 + t) * H + h) * d + c] : p.decay_out[(row0 + t) * H + h];
+                rg[e][j] = CHANNEL ? p.decay_out[(int64_t)((row0 + t) * H + h) * d + c] : p.decay_out[(row0 + t) * H + h];
             }
         }
         if (tid < TT * COLS) {
             int t = tid / COLS, jj = j0 + tid % COLS;
             t = t < nt ? t : nt - 1;
             jj = jj < dv ? jj : dv - 1;
-            rv = p.rows_in[(row0 + t) * p.row_stride + p.v_off + h * dv + jj];
+            rv = p.rows_in[(int64_t)(row0 + t) * stride + p.v_off + h * dv + jj];
         }
         if (tid < TT * 8) {
             int t = tid >> 3;
             t = t < nt ? t : nt - 1;
-            rcoef = p.coef[((row0 + t) * H + h) * 8 + (tid & 7)];
+            rcoef = p.coef[(int64_t)((row0 + t) * H + h) * 8 + (tid & 7)];
         }
     };
     auto place = [&](int tile) {
@@ -275,7 +295,7 @@ __global__ void __launch_bounds__(2 * THREADS) gated_delta_scan_kernel(GatedDelt
 #pragma unroll
         for (int i = 0; i < RC; i++)
 #pragma unroll
-            for (int c = 0; c < CW; c++) st[i][c] = sm.st[channel(i)][warp * CW + c];
+            for (int c = 0; c < CW; c++) st[i][c] = sm.st[channel(i)][warp * CW + (c ^ mine_c)];
     }
     for (int tile = 0; tile < tiles; tile++) {
         if (stages) {
@@ -294,8 +314,8 @@ __global__ void __launch_bounds__(2 * THREADS) gated_delta_scan_kernel(GatedDelt
 #pragma unroll
                     for (int i = 0; i < RC; i += V) {
                         float k4[V], q4[V];
-                        lds<V>(&in.gk[ch * C + j][channel(i)], k4);
-                        lds<V>(&in.gq[ch * C + j][channel(i)], q4);
+                        lds<V>(&in.gk[ch * C + (j ^ mine_t)][channel(i)], k4);
+                        lds<V>(&in.gq[ch * C + (j ^ mine_t)][channel(i)], q4);
 #pragma unroll
                         for (int w = 0; w < V; w++)
 #pragma unroll
@@ -305,23 +325,22 @@ __global__ void __launch_bounds__(2 * THREADS) gated_delta_scan_kernel(GatedDelt
                             }
                     }
                 }
-                const float t1 = add_over_lanes<NV, 16>(a1, lane);
+                // what a token writes but for its four's earlier writes: the lane that has the sum takes it off the value
+                const float t1 = in.v[ch * C + mine_t][warp * CW + mine_c] - fold_lanes<NV, 16>(a1);
                 float u[C][CW];
 #pragma unroll
                 for (int j = 0; j < C; j++)
 #pragma unroll
-                    for (int c = 0; c < CW; c++) u[j][c] = __shfl_sync(0xffffffffu, t1, (j * CW + c) * PER);
-                const float t2 = add_over_lanes<NV, 16>(a2, lane);
-                if (lane % PER == 0) sm.p2[tile & 1][ch * C + lane / PER / CW][warp * CW + lane / PER % CW] = t2;
+                    for (int c = 0; c < CW; c++) u[j][c] = __shfl_sync(0xffffffffu, t1, (8 * j + PER * c) ^ (PER * mine_c));
+                const float t2 = fold_lanes<NV, 16>(a2);
+                if (lane % PER == 0) sm.p2[tile & 1][ch * C + mine_t][warp * CW + mine_c] = t2;
 #pragma unroll
                 for (int j = 0; j < C; j++) {
                     const float4 a4 = *reinterpret_cast<const float4*>(&sm.coef[tile & 3][ch * C + j][0]);
                     const float aa[C - 1] = {a4.x, a4.y, a4.z};
-                    float vj[CW];
-                    lds<CW>(&in.v[ch * C + j][warp * CW], vj);
 #pragma unroll
                     for (int c = 0; c < CW; c++) {
-                        float t = vj[c] - u[j][c];
+                        float t = u[j][c];
 #pragma unroll
                         for (int s = 0; s < j; s++) t = fmaf(-aa[s], u[s][c], t);
                         u[j][c] = a4.w * t;
@@ -359,7 +378,7 @@ __global__ void __launch_bounds__(2 * THREADS) gated_delta_scan_kernel(GatedDelt
 #pragma unroll
         for (int i = 0; i < RC; i++)
 #pragma unroll
-            for (int c = 0; c < CW; c++) sm.st[channel(i)][warp * CW + c] = st[i][c];
+            for (int c = 0; c < CW; c++) sm.st[channel(i)][warp * CW + (c ^ mine_c)] = st[i][c];
     }
     __syncthreads();
     for (int idx = threadIdx.x; idx < D * COLS; idx += 2 * THREADS) {
@@ -510,13 +529,13 @@ int launch(const GatedDeltaParams& p, cudaStream_t stream) {
     if (!p.coef || !p.decay_out) GB_REFUSE("gated_delta: no room for the tokens' factors");
     gated_delta_prep_kernel<CHANNEL><<<dim3(ceil_div(p.max_q_len, C), ceil_div(p.heads, 4), p.nseq), 128, 0, stream>>>(p);
     GB_CHECK_LAUNCH("gated_delta_prep");
-    // few (head, column block) pairs: two columns a warp leave more CTAs, and warps, to hide one another's chains
-    const bool narrow = (int64_t)p.heads * p.nseq * ceil_div(p.dv, 16) < p.narrow_below;
+    // short heads and few (head, column block) pairs: two columns a warp leave more CTAs, and warps, to hide one another's chains
     const int rc = ceil_div(p.d, 32);
+    const bool narrow = rc <= 2 && (int64_t)p.heads * p.nseq * ceil_div(p.dv, 16) < p.narrow_below;
     if (rc <= 1) return narrow ? launch_scan<1, 2, CHANNEL>(p, stream) : launch_scan<1, 4, CHANNEL>(p, stream);
     if (rc <= 2) return narrow ? launch_scan<2, 2, CHANNEL>(p, stream) : launch_scan<2, 4, CHANNEL>(p, stream);
-    if (rc <= 4) return narrow ? launch_scan<4, 2, CHANNEL>(p, stream) : launch_scan<4, 4, CHANNEL>(p, stream);
-    return narrow ? launch_scan<8, 2, CHANNEL>(p, stream) : launch_scan<8, 4, CHANNEL>(p, stream);
+    if (rc <= 4) return launch_scan<4, 4, CHANNEL>(p, stream);
+    return launch_scan<8, 4, CHANNEL>(p, stream);
 }
 
 }  // namespace
@@ -528,6 +547,7 @@ GB_API int gb_gated_delta(const GatedDeltaParams* pp, cudaStream_t stream) {
         GB_REFUSE("gated_delta: %d heads over %d of %d key and %d value channels; at most 256 key channels", p.heads, p.kv_heads, p.d, p.dv);
     if (!p.rows_in || !p.decay_in || !p.beta_in || !p.a_log || !p.dt_bias || !p.state || !p.out) GB_REFUSE("gated_delta: a tensor is missing");
     if (p.head_stride < (int64_t)p.d * p.dv || p.slot_stride < p.head_stride * p.heads) GB_REFUSE("gated_delta: the state is too small for its heads");
+    if (p.row_stride > 0x7fffffff || (int64_t)p.rows * p.heads > 0x7fffffff) GB_REFUSE("gated_delta: %d rows of %d heads are too many for one launch", p.rows, p.heads);
     if (p.per_channel) return launch<true>(p, stream);
     return launch<false>(p, stream);
 }

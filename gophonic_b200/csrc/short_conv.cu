@@ -72,6 +72,25 @@ __device__ __forceinline__ void store_pair<__nv_bfloat16>(__nv_bfloat16* p, Pair
     if (n > 1) p[1] = __float2bfloat16_rn(v.b);
 }
 
+// two channels that are there, at an even place of an aligned row
+template <typename T>
+__device__ __forceinline__ Pair load_two(const T* p);
+template <>
+__device__ __forceinline__ Pair load_two<float>(const float* p) {
+    const float2 v = __ldg(reinterpret_cast<const float2*>(p));
+    return {v.x, v.y};
+}
+template <>
+__device__ __forceinline__ Pair load_two<__nv_bfloat16>(const __nv_bfloat16* p) {
+    const unsigned raw = __ldg(reinterpret_cast<const unsigned*>(p));
+    const __nv_bfloat162 v = *reinterpret_cast<const __nv_bfloat162*>(&raw);
+    return {__low2float(v), __high2float(v)};
+}
+
+__device__ __forceinline__ int64_t page_at(const ShortConvParams& p, int slot, int pos) {
+    return page_of(block_table_row(p.block_table, p.bt_stride, slot, p.max_slots), pos, p.bt_stride, p.pages);
+}
+
 // which head of the row: kind 0 q, 1 k, 2 v; c0 its first channel, n its width, at its number among its kind
 struct Head {
     int kind, c0, n, at;
@@ -84,9 +103,9 @@ __device__ __forceinline__ Head head_of(const ShortConvParams& p, int hh) {
 }
 
 // activation, rotation, norm and store of one row of one head, two channels a lane and piece.  CACHE: q into the buffer, k and v
-// into the cache (`bt`: the sequence's block-table row); else float32 rows.  HALF: channels i and i + rot / 2 may turn together
+// into the cache (`page`: the page of the row's position); else float32 rows.  HALF: channels i and i + rot / 2 may turn together
 template <typename T, int NE, bool CACHE, bool HALF>
-__device__ __forceinline__ void finish_head(const ShortConvParams& p, const Head& hd, int64_t row, int pos, const int* bt, Pair (&y)[NE], float* sh, int lane,
+__device__ __forceinline__ void finish_head(const ShortConvParams& p, const Head& hd, int64_t row, int pos, int64_t page, Pair (&y)[NE], float* sh, int lane,
                                             bool vec) {
     if (p.silu) {
 #pragma unroll
@@ -103,7 +122,7 @@ __device__ __forceinline__ void finish_head(const ShortConvParams& p, const Head
                 for (int e = 0; e < NE; e++) {
                     const int j = lane + 32 * e;       // channels 2j and 2j + 1
                     if (j < half) {
-                        const float c = ct[j], s = st[j];
+                        const float c = __ldg(ct + j), s = __ldg(st + j);
                         y[e] = {y[e].a * c - y[e].b * s, y[e].b * c + y[e].a * s};
                     }
                 }
@@ -145,7 +164,6 @@ __device__ __forceinline__ void finish_head(const ShortConvParams& p, const Head
     if constexpr (CACHE) {
         T* dst = (T*)p.out + row * p.out_stride + hd.c0;
         if (hd.kind != 0) {
-            const int64_t page = page_of(bt, pos, p.bt_stride, p.pages);
             const int heads = hd.kind == 1 ? p.k_heads : p.v_heads;
             dst = (T*)(hd.kind == 1 ? p.k_plane : p.v_plane) + ((page * heads + hd.at) * GB_PAGE + (pos % GB_PAGE)) * (int64_t)hd.n;
         }
@@ -199,7 +217,8 @@ __device__ __forceinline__ void convolve_row(const ShortConvParams& p, const Hea
     }
 }
 
-// Prompts of few taps: a warp's ROWS rows through a window of registers.  Rows whose taps all lie in their own portion, nearly
+// Prompts of few taps whose heads take two-channel accesses: a warp's ROWS rows through a window of registers, every load issued
+// ahead of the arithmetic (lanes beyond a narrower head repeat its last two channels and store nothing).  Rows whose taps all lie in their own portion, nearly
 // all of them, take straight code; a warp that holds a portion's first rows goes row by row.
 template <typename T, int ROWS, int TAPS, int NE, bool CACHE>
 __global__ void __launch_bounds__(32 * WARPS) short_conv_window_kernel(ShortConvParams p) {
@@ -211,18 +230,17 @@ __global__ void __launch_bounds__(32 * WARPS) short_conv_window_kernel(ShortConv
     const Head hd = head_of(p, hh);
     const int64_t r0 = (int64_t)blockIdx.x * ROWS;
     const int n = p.rows - r0 < ROWS ? (int)(p.rows - r0) : ROWS;
-    const bool vec = p.vec;
     const T* base = (const T*)p.src + hd.c0;
+    int at[NE];
+#pragma unroll
+    for (int e = 0; e < NE; e++) at[e] = min(2 * (lane + 32 * e), hd.n - 2);
     Pair x[ROWS + TAPS - 1][NE];
 #pragma unroll
     for (int i = 0; i < ROWS + TAPS - 1; i++) {
         int64_t r = r0 + i - (TAPS - 1);
         r = r < 0 ? 0 : (r < p.rows ? r : p.rows - 1);      // rows outside are not used
 #pragma unroll
-        for (int e = 0; e < NE; e++) {
-            const int c = 2 * (lane + 32 * e);
-            x[i][e] = load_pair<T>(base + r * p.row_stride + c, min(2, hd.n - c), vec);
-        }
+        for (int e = 0; e < NE; e++) x[i][e] = load_two<T>(base + r * p.row_stride + at[e]);
     }
     const int seq0 = p.row_seq[r0];
     const bool plain = p.row_seq[r0 + n - 1] == seq0 && r0 - p.seq_q_start[seq0] >= TAPS - 1;
@@ -233,29 +251,34 @@ __global__ void __launch_bounds__(32 * WARPS) short_conv_window_kernel(ShortConv
             int slot = p.seq_slot[seq];
             if (!gb_check(slot, p.max_slots, GB_CHECK_SLOT)) slot = 0;
             Pair y[NE];
-            convolve_row<T, NE>(p, hd, row, (int)(row - p.seq_q_start[seq]), slot, y, lane, vec);
-            finish_head<T, NE, CACHE, false>(p, hd, row, CACHE || p.rot > 0 ? p.row_pos[row] : 0,
-                                             CACHE ? block_table_row(p.block_table, p.bt_stride, slot, p.max_slots) : nullptr, y, nullptr, lane, vec);
+            convolve_row<T, NE>(p, hd, row, (int)(row - p.seq_q_start[seq]), slot, y, lane, true);
+            const int pos = CACHE || p.rot > 0 ? p.row_pos[row] : 0;
+            finish_head<T, NE, CACHE, false>(p, hd, row, pos, CACHE && hd.kind != 0 ? page_at(p, slot, pos) : 0, y, nullptr, lane, true);
         }
         return;
     }
     Pair w[TAPS][NE];
 #pragma unroll
     for (int e = 0; e < NE; e++) {
-        const int c = 2 * (lane + 32 * e), m = min(2, hd.n - c);
 #pragma unroll
         for (int j = 0; j < TAPS; j++) {
             w[j][e] = {1.f, 1.f};
-            if (p.conv_w) w[j][e] = load_pair<float>(p.conv_w + (int64_t)j * p.channels + hd.c0 + c, m, vec);
+            if (p.conv_w) w[j][e] = load_two<float>(p.conv_w + (int64_t)j * p.channels + hd.c0 + at[e]);
+            if (2 * (lane + 32 * e) >= hd.n) w[j][e] = {0.f, 0.f};      // a lane beyond the head has zeros
         }
         if (p.bias) {
-            const Pair bias = load_pair<float>(p.bias + hd.c0 + c, m, vec);
+            const Pair bias = load_two<float>(p.bias + hd.c0 + at[e]);
 #pragma unroll
             for (int i = 0; i < ROWS + TAPS - 1; i++) x[i][e] = {x[i][e].a + bias.a, x[i][e].b + bias.b};
         }
     }
     const int pos0 = CACHE || p.rot > 0 ? p.row_pos[r0] : 0;      // rows of a sequence are consecutive positions
-    const int* bt = CACHE ? block_table_row(p.block_table, p.bt_stride, p.seq_slot[seq0], p.max_slots) : nullptr;
+    int64_t first_page = 0, last_page = 0;                        // eight rows lie in two pages at most
+    if (CACHE && hd.kind != 0) {
+        const int slot = p.seq_slot[seq0];
+        first_page = page_at(p, slot, pos0);
+        last_page = page_at(p, slot, pos0 + n - 1);
+    }
 #pragma unroll
     for (int i = 0; i < ROWS; i++) {
         if (i >= n) break;
@@ -266,7 +289,7 @@ __global__ void __launch_bounds__(32 * WARPS) short_conv_window_kernel(ShortConv
 #pragma unroll
             for (int j = 0; j < TAPS; j++) y[e] = {fmaf(w[j][e].a, x[i + j][e].a, y[e].a), fmaf(w[j][e].b, x[i + j][e].b, y[e].b)};
         }
-        finish_head<T, NE, CACHE, false>(p, hd, r0 + i, pos0 + i, bt, y, nullptr, lane, vec);
+        finish_head<T, NE, CACHE, false>(p, hd, r0 + i, pos0 + i, (pos0 + i) / GB_PAGE == pos0 / GB_PAGE ? first_page : last_page, y, nullptr, lane, true);
     }
 }
 
@@ -286,8 +309,8 @@ __global__ void __launch_bounds__(32 * WARPS) short_conv_row_kernel(ShortConvPar
     if (!gb_check(slot, p.max_slots, GB_CHECK_SLOT)) slot = 0;
     Pair y[NE];
     convolve_row<T, NE>(p, hd, row, (int)(row - p.seq_q_start[seq]), slot, y, lane, p.vec);
-    finish_head<T, NE, CACHE, true>(p, hd, row, CACHE || p.rot > 0 ? p.row_pos[row] : 0,
-                                    CACHE ? block_table_row(p.block_table, p.bt_stride, slot, p.max_slots) : nullptr, y, sh[warp], lane, p.vec);
+    const int pos = CACHE || p.rot > 0 ? p.row_pos[row] : 0;
+    finish_head<T, NE, CACHE, true>(p, hd, row, pos, CACHE && hd.kind != 0 ? page_at(p, slot, pos) : 0, y, sh[warp], lane, p.vec);
 }
 
 // the last taps - 1 rows u of every sequence's portion into its state; a portion shorter than that pushes the older rows on
@@ -318,7 +341,7 @@ int launch_ne(const ShortConvParams& p, cudaStream_t stream) {
     const int heads = p.q_heads + p.k_heads + p.v_heads;
     const int hy = ceil_div(heads, WARPS);
     if (hy > 65535) GB_REFUSE("short_conv: %d heads exceed one launch", heads);
-    if (p.max_q_len != 1 && p.taps <= 4 && p.rows >= WINDOW_MIN_ROWS && (p.rot == 0 || p.pairs)) {
+    if (p.max_q_len != 1 && p.taps <= 4 && p.rows >= WINDOW_MIN_ROWS && p.vec && (p.rot == 0 || p.pairs)) {
         const dim3 grid(ceil_div(p.rows, WINDOW_ROWS), hy), block(32 * WARPS);
         switch (p.taps) {
             case 1: launch_pdl(short_conv_window_kernel<T, WINDOW_ROWS, 1, NE, CACHE>, grid, block, 0, stream, p); break;

@@ -1855,7 +1855,7 @@ class _GatedDeltaParams(Structure):
     ]
 
 
-GATED_DELTA_NARROW = 296     # fewer (head, 16 value columns) pairs than this: two columns a warp, twice the CTAs
+GATED_DELTA_NARROW = 296     # heads of up to 64 key channels, fewer (head, 16 value columns) pairs than this: two columns a warp, twice the CTAs
 
 
 def gated_delta(qkv: torch.Tensor, heads: int, kv_heads: int, d: int, dv: int, decay: torch.Tensor, dt_bias: torch.Tensor, a_log: torch.Tensor,
