@@ -19,7 +19,7 @@
 // Columns of S are independent of one another, so the work is spread over (sequence, head, block of value columns).  A warp
 // owns CW columns, its 32 lanes the key channels (RC each); a thread keeps RC x CW state elements in registers across the
 // step.  The four tokens' partial sums a lane are added over the lanes by halving the values and the lanes; the 4 x CW finished
-// v - S^T (G k) are then broadcast and every lane solves the four small triangular systems itself.  A prompt of one sequence leaves
+// v - S^T (G k) then pass through shared memory to all lanes, and every lane solves the four small triangular systems itself.  A prompt of one sequence leaves
 // every scheduler one such warp, so nothing but this chain is on it: four further warps of the CTA fetch the tokens' rows, form
 // the products of decays and lay them out in shared memory a tile of eight tokens ahead, and add the outputs' remaining terms a
 // tile behind.
@@ -125,20 +125,15 @@ __global__ void __launch_bounds__(128) gated_delta_prep_kernel(GatedDeltaParams 
     }
 }
 
-// The same for lanes that hold their values in an order of their own: the values of numbers N / 2 .. N - 1 are the ones the lane O
-// away keeps, so nothing is chosen.
-template <int N, int O>
-__device__ __forceinline__ float fold_lanes(float* a) {
-    if constexpr (O == 0) {
-        return a[0];
-    } else if constexpr (N == 1) {
-        a[0] += __shfl_xor_sync(0xffffffffu, a[0], O);
-        return fold_lanes<1, O / 2>(a);
-    } else {
+// The same for 4 N values in an order of the lane's own over the first two steps: the values of the upper half are the ones the
+// lane O away keeps, so nothing is chosen there.
+template <int N>
+__device__ __forceinline__ float fold_lanes(float* a, int lane) {
 #pragma unroll
-        for (int j = 0; j < N / 2; j++) a[j] += __shfl_xor_sync(0xffffffffu, a[j + N / 2], O);
-        return fold_lanes<N / 2, O / 2>(a);
-    }
+    for (int j = 0; j < 2 * N; j++) a[j] += __shfl_xor_sync(0xffffffffu, a[j + 2 * N], 16);
+#pragma unroll
+    for (int j = 0; j < N; j++) a[j] += __shfl_xor_sync(0xffffffffu, a[j + N], 8);
+    return add_over_lanes<N, 4>(a, lane);
 }
 
 template <int V>
@@ -173,6 +168,7 @@ struct ScanShared {
     } tile[2];
     float u[2][TT][COLS], p2[2][TT][COLS];
     float coef[4][TT][8];
+    float left[WARPS][2][C][CW];      // a warp's finished v - S^T (G k), for its lanes
     float st[D][COLS + 1];
 };
 
@@ -196,8 +192,8 @@ __global__ void __launch_bounds__(2 * THREADS) gated_delta_scan_kernel(GatedDelt
     if (!gb_check(slot, p.max_slots, GB_CHECK_SLOT)) slot = 0;
     float* S = p.state + (int64_t)slot * p.slot_stride + (int64_t)h * p.head_stride;
     auto channel = [&](int i) { return i / V * (32 * V) + lane * V + i % V; };
-    // A thread's slot j of the four tokens' sums is token j ^ mine_t and its column slot c is column c ^ mine_c of the warp's, so that
-    // adding over the lanes (fold_lanes) leaves each lane the sum of token mine_t and column mine_c: lane 8 j + PER c has (j, c)
+    // A thread's slot j of the four tokens' sums is token j ^ mine_t; adding over the lanes (fold_lanes) leaves each lane the sum of
+    // token mine_t and column mine_c
     const int mine_t = lane >> 3, mine_c = (lane / PER) % CW;
     const int tiles = (q_len + TT - 1) / TT;
 
@@ -295,7 +291,7 @@ __global__ void __launch_bounds__(2 * THREADS) gated_delta_scan_kernel(GatedDelt
 #pragma unroll
         for (int i = 0; i < RC; i++)
 #pragma unroll
-            for (int c = 0; c < CW; c++) st[i][c] = sm.st[channel(i)][warp * CW + (c ^ mine_c)];
+            for (int c = 0; c < CW; c++) st[i][c] = sm.st[channel(i)][warp * CW + c];
     }
     for (int tile = 0; tile < tiles; tile++) {
         if (stages) {
@@ -326,13 +322,13 @@ __global__ void __launch_bounds__(2 * THREADS) gated_delta_scan_kernel(GatedDelt
                     }
                 }
                 // what a token writes but for its four's earlier writes: the lane that has the sum takes it off the value
-                const float t1 = in.v[ch * C + mine_t][warp * CW + mine_c] - fold_lanes<NV, 16>(a1);
+                const float t1 = in.v[ch * C + mine_t][warp * CW + mine_c] - fold_lanes<CW>(a1, lane);
+                if (lane % PER == 0) sm.left[warp][ch & 1][mine_t][mine_c] = t1;
+                __syncwarp();
                 float u[C][CW];
 #pragma unroll
-                for (int j = 0; j < C; j++)
-#pragma unroll
-                    for (int c = 0; c < CW; c++) u[j][c] = __shfl_sync(0xffffffffu, t1, (8 * j + PER * c) ^ (PER * mine_c));
-                const float t2 = fold_lanes<NV, 16>(a2);
+                for (int j = 0; j < C; j++) lds<CW>(sm.left[warp][ch & 1][j], u[j]);
+                const float t2 = fold_lanes<CW>(a2, lane);
                 if (lane % PER == 0) sm.p2[tile & 1][ch * C + mine_t][warp * CW + mine_c] = t2;
 #pragma unroll
                 for (int j = 0; j < C; j++) {
@@ -378,7 +374,7 @@ __global__ void __launch_bounds__(2 * THREADS) gated_delta_scan_kernel(GatedDelt
 #pragma unroll
         for (int i = 0; i < RC; i++)
 #pragma unroll
-            for (int c = 0; c < CW; c++) sm.st[channel(i)][warp * CW + (c ^ mine_c)] = st[i][c];
+            for (int c = 0; c < CW; c++) sm.st[channel(i)][warp * CW + c] = st[i][c];
     }
     __syncthreads();
     for (int idx = threadIdx.x; idx < D * COLS; idx += 2 * THREADS) {
