@@ -688,7 +688,7 @@ def probe(name, **opts):
             work = rows * W * (2 + 4)
             fn = lambda: ops.short_conv(src, out, kvh, kvh, heads, d, d, conv, state, packed, silu=True, norm=ops.HEAD_NORM_UNIT, eps=1e-6, q_scale=0.1)
         unit = "GB/s"
-    elif name in ("sandwich_mid", "sandwich_open_4", "sandwich_open_8", "norm_scale_add_rows", "conv_rows_prompt", "conv_qkv_prompt"):
+    elif name in ("sandwich_mid", "sandwich_pair", "sandwich_open_4", "sandwich_open_8", "norm_scale_add_rows", "conv_rows_prompt", "conv_qkv_prompt"):
         # row-wise kernels over 16384 rows of 2048 (each operand is as large as L2): a sublayer's output joined and normed; the
         # same with a weighted sum over 4 or 8 planes; the postnorm block's kernel; the convolutions ahead of a mixer
         from types import SimpleNamespace
@@ -709,6 +709,10 @@ def probe(name, **opts):
             result = torch.empty_like(base)
             work = rows * W * (4 + 4 + 4 + 2)
             fn = lambda: ops.sandwich_rows(base=base, y=y, y_weight=w, y_eps=1e-6, result=result, out=x, norm_weight=w, eps=1e-6)
+        elif name == "sandwich_pair":      # a sublayer that left two outputs
+            result, second = torch.empty_like(base), f32(rows, W)
+            work = rows * W * (4 + 4 + 4 + 4 + 2)
+            fn = lambda: ops.sandwich_rows(base=base, y=y, y_weight=w, y_eps=1e-6, result=result, out=x, norm_weight=w, eps=1e-6, pair=(second, w, w, 1e-6))
         elif name.startswith("sandwich_open"):
             n = int(name.rsplit("_", 1)[1])
             planes, avg, x_out, normed = f32(n + 1, rows, W), torch.ones(n + 1, device=dev), torch.empty_like(base), torch.empty_like(base)
