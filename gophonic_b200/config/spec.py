@@ -124,8 +124,8 @@ class GatedAttentionSpec:
       behind the position encoding (only without a weight; with an encoding that keeps a head's length the two orders are
       the same function, since a rotation changes no sum of squares);
     * ``conv_taps`` > 0: a causal convolution over time on every channel of q, k and v directly behind the projection and its
-      bias, y_t = sum_j c[:, j] u_(t - taps + 1 + j), zeros before the sequence's start (tensors: the projection's name plus
-      ``conv_suffix``, [channels, taps]); a sequence's last taps - 1 projected rows are part of its state;
+      bias, y_t = sum_j c[:, j] u_(t - taps + 1 + j) with u zero ahead of the first token (tensors: the projection's name plus
+      ``conv_suffix``, [channels, taps]); the cache keeps taps - 1 projected rows a sequence for it;
     * ``value_from_key``: there is no value projection, the values are the keys as projected, before norm and rotation
       (``value_dim`` = ``head_dim``);
     * ``out_bias``: the output projection carries a bias too;
@@ -285,7 +285,7 @@ class DeltaRuleSpec:
 class GatedDeltaSpec:
     """The gated delta rule: per head a matrix state S (key_dim x value_dim, float32) with a decay g and a write strength b,
 
-        S <- diag(g) S,   u = b (v - S^T k),   S <- S + k u^T,   o = S^T q      (the read-out sees the token's own write).
+        S <- diag(g) S,   u = b (v - S^T k),   S <- S + k u^T,   o = S^T q      (the write comes ahead of the read).
 
     q and k have ``kv_heads`` heads of key_dim (head h reads head h // (heads / kv_heads)), v ``heads`` of value_dim.  Each passes
     a short causal convolution over time per channel (``conv_taps``; 0: none; tensors: the projection's name plus ``conv_suffix``)
